@@ -579,6 +579,60 @@ int yalm_detokenize(const void *image, size_t size, const int *ids, int n, char 
 const char *yalm_error_string(int code);
 const char *yalm_version(void);
 
+/* ---- parallel blocks with one product in and one product out (csrc/ops_stack_block.cu) ----
+ * x = table[token] + bigram[row], row = (previous token * mul_prev + token * mul_cur) mod buckets, row `buckets` at position 0; also to
+ * x0 (NULL: not).  tokens (n) or, for n = 1, NULL and ctl[0]; prev: device word with the token before the call, replaced by its last. */
+int yalm_embed_bigram_rows(float *x, float *x0, const void *table, const void *bigram, int dtype, const int *tokens, int buckets, long long mul_prev,
+                           long long mul_cur, int *prev, int n, int dim, int pos0, const int *ctl, yalm_stream_t s);
+/* out[r] and / or out16[r] (bf16 if bf16 != 0, else fp16) = (x - mean) / sqrt(var + eps) * w + bias of row rows[r] (NULL: r), after
+ * x[row] += add[row] (add NULL: not).  bias optional. */
+int yalm_layer_norm_rows(float *out, void *out16, int bf16, float *x, const float *add, const int *rows, const float *w, const float *bias, float eps,
+                         int n, int dim, yalm_stream_t s);
+/* Slab i of out / out16 (n_mixes slabs of n x dim): h + (h of the previous position - h) mu[i], or h itself if bit i of plain_mask
+ * is set; mu (n_mixes, dim).  state (2, dim): row (position & 1) holds h of the last positions. */
+int yalm_mix_rows(float *out, void *out16, int bf16, const float *h, const float *mu, int n_mixes, int plain_mask, float *state, int n, int dim, int pos0,
+                  const int *ctl, yalm_stream_t s);
+/* in (n, ldi): projections q (kv_heads dim) | k | v (heads vdim); raw (n, ldi): beta (heads) | decay (heads) projections.  out (n, channels):
+ * silu of the causal convolution conv_w (channels, taps), q and k then x / sqrt(sum x^2 + unit_eps) per head, q also times q_scale;
+ * gates (n, 2 heads): exp(-exp(a_log) softplus(decay + dt_bias)) | sigmoid(beta).  ring (taps, channels): inputs by position % taps. */
+int yalm_delta_in_rows(float *out, float *gates, const float *in, const float *raw, int ldi, const float *conv_w, float *ring, const float *a_log,
+                       const float *dt_bias, int n, int heads, int kv_heads, int dim, int vdim, int taps, float unit_eps, float q_scale, int pos0,
+                       const int *ctl, yalm_stream_t s);
+/* out[m, c] = exp(-exp(w0[c] + w2[c] . tanh(t[m]))), w2 (channels, rank) in `dtype`. */
+int yalm_wkv_decay_rows(float *out, int ldo, const float *t, int ldt, const void *w2, const float *w0, int dtype, int n, int channels, int rank,
+                        yalm_stream_t s);
+/* out[m, h, :] = (M + diag(bonus[h]) k v^T)^T q, then M <- diag(decay) M + k v^T; k, q, decay (n, heads D), v, out (n, heads P), bonus
+ * (heads, D), state (heads, P, D).  D <= 256. */
+int yalm_state_scan_bonus_rows(float *out, int ldo, const float *k, int ldk, const float *q, int ldq, const float *v, int ldv, const float *decay, int ldd,
+                               const float *bonus, float *state, int n, int heads, int D, int P, int pos0, const int *ctl, yalm_stream_t s);
+/* yalm_head_norm_rope_append_rows with biases (one per channel of all vectors; NULL: none) added first and, instead of the norm before
+ * the rotation, every query / key vector divided by its root mean square after it, without a weight. */
+int yalm_head_bias_rope_norm_append_rows(float *proj, int ld, int o_q, int o_k, int o_v, int n_q_vectors, int n_k_vectors, int n_v_heads, int dk, int dv,
+                                         const float *q_bias, const float *k_bias, const float *v_bias, const float *freq, float magnitude, int rot_dims,
+                                         int interleaved, float eps, void *key_ring, void *value_ring, int ring, int cache_f32, int n, int pos0,
+                                         const int *ctl, yalm_stream_t s);
+/* out / out16 (n, ldo): columns [0, heads vdim) = o, or per head o / sqrt(mean o^2 + eps) * norm_w[h * w_stride + c] * silu(gate) if norm_w;
+ * columns [heads vdim, + ff) = act(gu[f]) * gu[ff + f].  gate and gu rows have stride ldp. */
+int yalm_block_out_rows(float *out, void *out16, int bf16, int ldo, const float *o, int ldi, const float *gate, const float *gu, int ldp, const float *norm_w,
+                        int w_stride, float eps, int n, int heads, int vdim, int ff, int act, yalm_stream_t s);
+/* A decode row of a matrix-state mixer in one launch, from the row `proj` of the packed projection (o_*: offsets in it): what
+ * yalm_delta_in_rows / yalm_wkv_decay_rows, the scan and the per-head norm and gate of yalm_block_out_rows do. */
+int yalm_delta_step(float *out, float *state, const float *proj, int o_qkv, int o_gate, int o_beta, int o_decay, const float *conv_w, float *ring,
+                    const float *a_log, const float *dt_bias, const float *norm_w, int heads, int kv_heads, int dim, int vdim, int taps, float unit_eps,
+                    float q_scale, float eps, int pos0, const int *ctl, yalm_stream_t s);
+int yalm_wkv_step(float *out, float *state, const float *proj, int o_r, int o_k, int o_v, int o_gate, int o_decay, const void *w2, const float *w0,
+                  const float *bonus, const float *norm_w, int dtype, int heads, int dim, int rank, float eps, int pos0, const int *ctl, yalm_stream_t s);
+/* A decode row's products.  in: out (d) = W h, h the layer norm of x (norm_w, norm_b), by segments of output rows [segment_end[i - 1],
+ * segment_end[i]) blended with the previous position's h as in yalm_mix_rows (segment_end NULL: one segment; state NULL: nothing kept).
+ * out: res (d) += W [x1 (n1) | act(gu[f]) gu[ff + f]] (+ add).  Row lengths multiples of 8 (fp32: 4), 16-byte aligned. */
+int yalm_gemv_block_in(float *out, const float *x, const void *w, int n, int d, int dtype, const float *norm_w, const float *norm_b, float eps, int n_segments,
+                       const int *segment_end, const float *mu, int plain_mask, float *state, int pos0, const int *ctl, yalm_stream_t s);
+int yalm_gemv_block_out(float *res, const float *x1, int n1, const float *gu, int ff, int act, const void *w, int d, int dtype, const float *add,
+                        yalm_stream_t s);
+/* yalm_gemm_16 with one input per segment of output columns: a (n_segments M, K), segment bounds multiples of 4, the last one N. */
+int yalm_gemm_16_segments(float *c, int ldc, const void *a, const void *w, int M, int N, int K, int n_segments, const int *segment_end, int bf16,
+                          yalm_stream_t s);
+
 #ifdef __cplusplus
 }
 #endif

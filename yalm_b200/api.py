@@ -45,6 +45,9 @@ SYMBOLS = [
     "yalm_attn_window_pool_sink", "yalm_attn_window_pool_mma_sink", "yalm_attn_latent_rows_sink", "yalm_head_norm_rope_append_rows", "yalm_diff_combine_rows",
     "yalm_act_rows", "yalm_token_side_rows", "yalm_token_side_gate_rows", "yalm_gemv_act_norm_residual_norm",
     "yalm_attn_latent_mma_shape", "yalm_attn_latent_mma_rows", "yalm_attn_latent_merge",
+    "yalm_embed_bigram_rows", "yalm_layer_norm_rows", "yalm_mix_rows", "yalm_delta_in_rows", "yalm_wkv_decay_rows", "yalm_state_scan_bonus_rows",
+    "yalm_head_bias_rope_norm_append_rows", "yalm_block_out_rows", "yalm_delta_step", "yalm_wkv_step", "yalm_gemv_block_in", "yalm_gemv_block_out",
+    "yalm_gemm_16_segments",
     "yalm_tp_unique_id", "yalm_tp_init", "yalm_tp_finalize", "yalm_tp_shard_plan", "yalm_mega_tile_plan", "yalm_mega_attn_split", "yalm_mega_mma_plan", "yalm_mega_hb_share", "yalm_error_string", "yalm_version",
 ]
 

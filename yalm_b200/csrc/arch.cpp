@@ -153,8 +153,24 @@ int StackSpec::max_v_dim() const {
 int StackSpec::max_o_dim() const {
 	int m = 0;
 	for (const LayerSpec &l : layers)
-		m = std::max({m, l.mix.heads * l.mix.maps * l.mix.vdim, l.ssm.inner(), l.delta.heads * l.delta.vdim, l.mix.heads * l.latent.kv_rank, l.gla.heads * l.gla.vdim});
+		m = std::max({m, l.mix.heads * l.mix.maps * l.mix.vdim, l.ssm.inner(), l.delta.heads * l.delta.vdim, l.mix.heads * l.latent.kv_rank, l.gla.heads * l.gla.vdim, l.wkv.inner()});
 	return m;
+}
+int StackSpec::max_block_out() const {
+	int m = 0;
+	for (const LayerSpec &l : layers) m = std::max(m, l.block_out_width());
+	return m;
+}
+std::vector<LayerRun> StackSpec::runs() const {
+	std::vector<LayerRun> out;
+	const int n = (int)layers.size();
+	auto span = [&](int a, int b, bool again) {
+		for (int i = a; i < b; ++i) out.push_back({i, again && i == a});
+	};
+	span(0, loop_stop, false);
+	for (int t = 1; t < loop_times; ++t) span(loop_start, loop_stop, true);
+	span(loop_stop, n, false);
+	return out;
 }
 int StackSpec::max_proj() const {
 	int m = 0;
@@ -178,6 +194,12 @@ int LayerSpec::proj_width() const {
 		return (latent.q_rank > 0 ? latent.q_rank : mix.heads * (mix.dim + latent.rot_dim)) + (latent.kv_from < 0 ? latent.kv_rank + latent.rot_dim : 0) +
 		       (mix.out_gate ? mix.heads * mix.vdim : 0);
 	if (kind == MixerKind::LinearAttention) return 2 * gla.heads * gla.dim + 2 * gla.heads * gla.vdim + gla.decay_rank;
+	// packed blocks (rows padded to a multiple of 8): the mixer's large projections, the feed-forward's gate and up, then what is not
+	// a multiple of anything
+	const int glu = ffn.kind == FfnSpec::Dense ? 2 * ffn.ff : 0;
+	if (kind == MixerKind::DeltaRule) return (2 * delta.kv_heads * delta.dim + 2 * delta.heads * delta.vdim + glu + 2 * delta.heads + 7) & ~7;
+	if (kind == MixerKind::TimeMix) return (4 * wkv.inner() + glu + wkv.decay_rank + 7) & ~7;
+	if (kind == MixerKind::Attention && mix.v_bias) return ((mix.heads + mix.kv_heads) * mix.dim + mix.kv_heads * mix.vdim + glu + 7) & ~7;
 	int n = mix.maps * (mix.heads + mix.kv_heads) * mix.dim + (mix.values_are_keys ? 0 : mix.kv_heads * mix.vdim) + (mix.out_gate ? mix.heads * mix.vdim : 0);
 	if (mix.head_gate) n = (n + mix.heads + 3) & ~3; // one gate column per head; rows stay 16-byte multiples
 	if (kind == MixerKind::Parallel) n += 2 * delta.kv_heads * delta.dim + delta.heads * delta.vdim + delta.heads + delta.decay_rank + delta.gate_rank;
@@ -186,16 +208,20 @@ int LayerSpec::proj_width() const {
 int LayerSpec::mixed_width() const {
 	if (kind == MixerKind::StateSpace) return ssm.inner();
 	if (kind == MixerKind::LinearAttention) return gla.heads * gla.vdim;
+	if (kind == MixerKind::DeltaRule) return delta.heads * delta.vdim;
+	if (kind == MixerKind::TimeMix) return wkv.inner();
 	return mix.heads * mix.vdim + (kind == MixerKind::Parallel ? delta.heads * delta.vdim : 0);
 }
 int LayerSpec::conv_width() const {
 	if (kind == MixerKind::StateSpace) return ssm.conv_channels();
 	if (kind == MixerKind::LatentAttention) return mix.heads * (mix.dim + latent.rot_dim); // the queries as projected
-	return kind == MixerKind::Parallel ? 2 * delta.kv_heads * delta.dim + delta.heads * delta.vdim : 0;
+	return kind == MixerKind::Parallel || kind == MixerKind::DeltaRule ? delta.conv_channels() : 0;
 }
 int LayerSpec::aux_width() const {
 	if (kind == MixerKind::LatentAttention) return mix.heads * (latent.kv_rank + latent.rot_dim); // the queries against the cached rows
 	if (kind == MixerKind::LinearAttention) return gla.heads * gla.dim;                       // the decays
+	if (kind == MixerKind::DeltaRule) return 2 * delta.heads;                                                          // decay, beta
+	if (kind == MixerKind::TimeMix) return wkv.inner();                                                                // the decays
 	return kind == MixerKind::Parallel ? delta.heads * delta.dim + delta.heads * delta.vdim : 0;
 }
 int StackSpec::max_ff() const {
@@ -206,12 +232,22 @@ int StackSpec::max_ff() const {
 
 void RotarySpec::table(std::vector<float> *freqs, float *magnitude) const {
 	const int half = dims / 2;
+	const double pi = 3.14159265358979323846;
 	freqs->assign(half, 0.f);
 	*magnitude = 1.f;
 	std::vector<double> f(half);
 	for (int i = 0; i < half; ++i) f[i] = std::pow(base, -2.0 * i / dims);
-	if (factor > 0.0) {
-		const double pi = 3.14159265358979323846;
+	if (factor > 0.0 && high > 0.0) {
+		for (double &fi : f) {
+			const double wave = 2.0 * pi / fi;
+			if (wave < original / high) continue;
+			if (wave > original / low) fi /= factor;
+			else {
+				const double s = (original / wave - low) / (high - low);
+				fi = (1.0 - s) * fi / factor + s * fi;
+			}
+		}
+	} else if (factor > 0.0) {
 		auto at = [&](double turns) { return dims * std::log(original / (2.0 * pi * turns)) / (2.0 * std::log(base)); };
 		const double lo = std::max(std::floor(at(fast)), 0.0), hi = std::min(std::ceil(at(slow)), (double)(dims - 1));
 		for (int i = 0; i < half; ++i) {
@@ -811,11 +847,167 @@ int configure_kiduvik(const JValue &j, Config &cfg) {
 	return 0;
 }
 
+// ---- Fafelix ---------------------------------------------------------------------------------------------------------
+// A decoder-only stack of parallel blocks, x <- x + (mixer(h) + ff(h)) with ONE layer norm (weight and bias) h = N(x) per layer; a
+// bigram table is added to the token embedding, and a span of layers may run several times in a row with the same weights,
+// every pass with its own caches and state and, after the first, with the embedding output added before it.  Mixers: a gated
+// delta rule with one decay per head behind short convolutions; causal attention with biased projections, interleaved rotary
+// positions rescaled by wavelength, a weightless RMS norm of q and k after the rotation, grouped key / value heads and a stored sink
+// per head; time mixing (five blends with the previous token's h, a decay per key channel, a bonus for the current token).
+// Feed-forward: dense, SiLU-gated.
+std::string fafelix_tensor(int layer, TensorRole role, int) {
+	const std::string l = "l" + std::to_string(layer) + ".", m = l + "mix.", f = l + "mlp.";
+	switch (role) {
+	case TensorRole::Embed: return "embed";
+	case TensorRole::Bigram: return "bigram";
+	case TensorRole::FinalNorm: return "final.norm";
+	case TensorRole::FinalNormBias: return "final.norm.b";
+	case TensorRole::Head: return "head";
+	case TensorRole::Norm1: return l + "norm1";
+	case TensorRole::Norm1Bias: return l + "norm1.b";
+	case TensorRole::Wq: return m + "q";
+	case TensorRole::Wk: return m + "k";
+	case TensorRole::Wv: return m + "v";
+	case TensorRole::Wo: return m + "o";
+	case TensorRole::QBias: return m + "q.b";
+	case TensorRole::KBias: return m + "k.b";
+	case TensorRole::VBias: return m + "v.b";
+	case TensorRole::Sink: return m + "sink";
+	case TensorRole::DeltaQ: return m + "q";
+	case TensorRole::DeltaK: return m + "k";
+	case TensorRole::DeltaV: return m + "v";
+	case TensorRole::DeltaQConv: return m + "q.conv";
+	case TensorRole::DeltaKConv: return m + "k.conv";
+	case TensorRole::DeltaVConv: return m + "v.conv";
+	case TensorRole::DeltaBeta: return m + "b";
+	case TensorRole::DeltaDecay: return m + "a";
+	case TensorRole::DeltaALog: return m + "A_log";
+	case TensorRole::DeltaDtBias: return m + "dt_bias";
+	case TensorRole::DeltaNorm: return m + "norm";
+	case TensorRole::DeltaGate: return m + "g";
+	case TensorRole::WkvR: return m + "r";
+	case TensorRole::OutGate: return m + "g";
+	case TensorRole::WkvMuR: return m + "mu.r";
+	case TensorRole::WkvMuK: return m + "mu.k";
+	case TensorRole::WkvMuV: return m + "mu.v";
+	case TensorRole::WkvMuG: return m + "mu.g";
+	case TensorRole::WkvMuW: return m + "mu.w";
+	case TensorRole::WkvDecay1: return m + "w1";
+	case TensorRole::WkvDecay2: return m + "w2";
+	case TensorRole::WkvDecayBias: return m + "w0";
+	case TensorRole::WkvBonus: return m + "u";
+	case TensorRole::WkvNorm: return m + "norm";
+	case TensorRole::Gate: return f + "gate";
+	case TensorRole::Up: return f + "up";
+	case TensorRole::Down: return f + "down";
+	default: break;
+	}
+	return "";
+}
+
+int fail_fafelix(const char *what) {
+	fprintf(stderr, "yalm_b200: Fafelix config.json: %s\n", what);
+	return YALM_EFORMAT;
+}
+
+// No table bounds the context (rotary positions, recurrent state): the key / value rings of the causal layers are sized by the
+// context the caller asks for, else by "max_positions", else by this.
+constexpr int kFafelixContext = 32768;
+
+int configure_fafelix(const JValue &j, Config &cfg) {
+	auto spec = std::make_shared<StackSpec>();
+	StackSpec &s = *spec;
+	s.arch = "Fafelix";
+	s.width = j["width"].integer(0);
+	s.vocab = j["vocab"].integer(0);
+	s.max_positions = j["max_positions"].integer(kFafelixContext);
+	s.norm_eps = (float)j["norm"]["eps"].number(1e-5);
+	s.layer_norm = s.norm_bias = true;
+	s.parallel_block = s.packed_block = true;
+	s.tensor_name = fafelix_tensor;
+	if (s.width < 1 || s.vocab < 1 || s.max_positions < 1) return fail_fafelix("width and vocab must be positive");
+	const JValue &big = j["embedding"]["bigram"];
+	if (big.is_object()) {
+		s.bigram.buckets = big["buckets"].integer(0);
+		s.bigram.mul_prev = (long long)big["mul_prev"].number(0.0), s.bigram.mul_cur = (long long)big["mul_cur"].number(0.0);
+		if (s.bigram.buckets < 1) return fail_fafelix("embedding.bigram.buckets must be positive");
+	}
+	const JValue &layers = j["layers"];
+	if (!layers.is_array() || layers.arr.empty()) return fail_fafelix("'layers' must be a non-empty list");
+	for (const JValue &jl : layers.arr) {
+		LayerSpec L;
+		const std::string type = jl["type"].string_or("");
+		const JValue &m = jl["mixer"];
+		if (type == "delta") {
+			L.kind = MixerKind::DeltaRule;
+			DeltaSpec &d = L.delta;
+			d.heads = m["heads"].integer(0), d.kv_heads = m["kv_heads"].integer(d.heads);
+			d.dim = m["dim"].integer(0), d.vdim = m["vdim"].integer(d.dim), d.conv = m["conv"].integer(0);
+			d.head_decay = d.full_gate = true;
+			if (d.heads < 1 || d.kv_heads < 1 || d.heads % d.kv_heads || d.dim < 1 || d.vdim < 1 || d.conv < 1) return fail_fafelix("bad delta-rule sizes");
+		} else if (type == "attention") {
+			L.kind = MixerKind::Attention;
+			MixerSpec &x = L.mix;
+			x.heads = m["heads"].integer(0), x.kv_heads = m["kv_heads"].integer(x.heads);
+			x.dim = m["dim"].integer(0), x.vdim = m["vdim"].integer(x.dim);
+			x.scale = (float)m["scale"].number(1.0);
+			x.qk_bias = x.v_bias = x.sink = true;
+			x.qk_norm = QkNorm::PerHeadRotated;
+			const JValue &r = m["rot"], &sc = r["scaling"];
+			x.rot.dims = r["dims"].integer(0), x.rot.base = r["base"].number(10000.0), x.rot.interleaved = true;
+			if (sc.is_object()) {
+				x.rot.factor = sc["factor"].number(0.0), x.rot.original = sc["original"].number(0.0);
+				x.rot.low = sc["low"].number(0.0), x.rot.high = sc["high"].number(0.0);
+				if (!(x.rot.factor > 0.0) || !(x.rot.original > 0.0) || !(x.rot.low > 0.0) || !(x.rot.high > x.rot.low)) return fail_fafelix("bad rotary scaling");
+			}
+			if (x.heads < 1 || x.kv_heads < 1 || x.heads % x.kv_heads || x.dim < 1 || x.vdim < 1) return fail_fafelix("bad attention sizes");
+			if (x.rot.dims < 0 || x.rot.dims % 2 || x.rot.dims > x.dim || !(x.rot.base > 0.0)) return fail_fafelix("rot.dims must be even and at most dim");
+		} else if (type == "wkv") {
+			L.kind = MixerKind::TimeMix;
+			L.wkv.heads = m["heads"].integer(0), L.wkv.dim = m["dim"].integer(0);
+			if (L.wkv.heads < 1 || L.wkv.dim < 1) return fail_fafelix("bad time-mixing sizes");
+		} else
+			return fail_fafelix("unknown layer type (this build has: delta, attention, wkv)");
+		const JValue &f = jl["mlp"];
+		if (f.is_object()) {
+			if (f["kind"].string_or("") != "dense") return fail_fafelix("unknown mlp kind (this build has: dense)");
+			L.ffn.kind = FfnSpec::Dense, L.ffn.act = GluAct::Silu;
+			L.ffn.ff = f["ff"].integer(0);
+			if (L.ffn.ff < 1) return fail_fafelix("bad feed-forward size");
+		}
+		s.layers.push_back(L);
+	}
+	const JValue &loop = j["loop"];
+	if (loop.is_object()) {
+		s.loop_start = loop["start"].integer(0), s.loop_stop = loop["stop"].integer(0), s.loop_times = loop["times"].integer(1);
+		if (s.loop_start < 0 || s.loop_stop <= s.loop_start || s.loop_stop > (int)s.layers.size() || s.loop_times < 1) return fail_fafelix("bad loop");
+	}
+	cfg.stack = spec;
+	cfg.dim = s.width;
+	cfg.vocab_size = s.vocab;
+	cfg.n_layers = (int)s.layers.size();
+	cfg.max_seq_len = s.max_positions;
+	cfg.norm_eps = s.norm_eps;
+	cfg.hidden_dim = std::max(1, s.max_ff());
+	cfg.n_heads = cfg.n_kv_heads = 1;
+	for (const LayerSpec &l : s.layers)
+		if (l.kind == MixerKind::Attention) {
+			cfg.n_heads = l.mix.heads, cfg.n_kv_heads = l.mix.kv_heads;
+			break;
+		}
+	cfg.head_dim = 8;
+	while (cfg.n_heads * cfg.head_dim < std::max({s.max_aux(), s.max_o_dim(), s.max_q_dim()})) cfg.head_dim *= 2;
+	cfg.rotary_dim = 0;
+	cfg.n_experts = 0, cfg.n_experts_active = 0;
+	return 0;
+}
+
 const ArchEntry kArchs[] = {
     {"Retezen", configure_retezen},
     {"Fapudra", configure_fapudra},
     {"Fegizen", configure_fegizen},
     {"Kiduvik", configure_kiduvik},
+    {"Fafelix", configure_fafelix},
 };
 
 } // namespace

@@ -19,7 +19,8 @@ namespace yalm {
 enum class QkNorm {
 	None,
 	WholeProjection, /* RMS over all heads' channels at once, one weight per channel */
-	PerHead          /* RMS over each head's dim channels (each map's, with several maps), one weight of size dim shared by all heads */
+	PerHead,         /* RMS over each head's dim channels (each map's, with several maps), one weight of size dim shared by all heads */
+	PerHeadRotated   /* RMS over each head's dim channels after the rotation, no weight */
 };
 // Gated feed-forward activations: y = act(g) * (u + up_offset), with optional clamps on g (from above) and u (both sides).
 enum class GluAct {
@@ -37,7 +38,9 @@ enum class MixerKind {
 	StateSpace, // SsmSpec: a selective state-space recurrence with a scalar decay per head
 	Parallel,   // two mixers side by side on the same input, added with fixed scales: attention (MixerSpec) + gated delta rule (DeltaSpec)
 	LatentAttention, // MixerSpec + LatentSpec: queries, keys and values through low-rank latents; the cache holds the key / value latent
-	LinearAttention  // GlaSpec: a (dim, vdim) matrix state per head with one decay per key channel
+	LinearAttention, // GlaSpec: a (dim, vdim) matrix state per head with one decay per key channel
+	DeltaRule,       // DeltaSpec alone
+	TimeMix          // WkvSpec: a matrix state with one decay per key channel, read out before the decay with a bonus for the current token
 };
 // How attention scores become weights.
 enum class AttnWeights { Softmax, Sigmoid /* sigmoid(score + head bias), not normalised over the keys */ };
@@ -46,12 +49,14 @@ enum class AttnWeights { Softmax, Sigmoid /* sigmoid(score + head bias), not nor
 // f_i = base^(-2 i / dims).  interleaved: pair i = channels (2 i, 2 i + 1); else (i, i + dims / 2).  factor > 0 rescales the
 // frequencies by wavelength (YaRN): with d(t) = dims ln(original / (2 pi t)) / (2 ln base), lo = max(floor(d(fast)), 0),
 // hi = min(ceil(d(slow)), dims - 1), r_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1): f_i <- f_i / factor * r_i + f_i (1 - r_i),
-// and cos and sin are multiplied by 0.1 ln(factor) + 1.
+// and cos and sin are multiplied by 0.1 ln(factor) + 1.  With high > 0 the rescaling is by two wavelength bounds instead (no
+// factor on cos and sin): a pair of wavelength l = 2 pi / f keeps f below original / high, takes f / factor above
+// original / low, and between them (1 - s) f / factor + s f with s = (original / l - low) / (high - low).
 struct RotarySpec {
 	int dims = 0;
 	double base = 10000.0;
 	bool interleaved = true;
-	double factor = 0.0, original = 0.0, fast = 0.0, slow = 0.0;
+	double factor = 0.0, original = 0.0, fast = 0.0, slow = 0.0, low = 0.0, high = 0.0;
 	// the table the kernels read: dims / 2 frequencies, and the factor on cos and sin (computed in double precision)
 	void table(std::vector<float> *freqs, float *magnitude) const;
 };
@@ -68,6 +73,7 @@ struct MixerSpec {
 	AttnWeights weights = AttnWeights::Softmax;
 	bool values_are_keys = false; // no value projection: v = k as projected (vdim == dim)
 	bool qk_bias = false;        // biases on the q and k projections
+	bool v_bias = false;         // a bias on the v projection
 	bool out_gate = false;       // heads * sigmoid(Wg input) before the output projection
 	int rel_rows = 0;            // > 0: a learned bias per (distance bucket, head) is added to the scaled score: distances below
 	int rel_far = 0;             // rel_rows / 2 have a row each, the rest are spaced logarithmically up to rel_far, then the last row
@@ -114,10 +120,23 @@ struct SsmSpec {
 // Gated delta rule with one decay per head and key channel: per head a (dim, vdim) matrix S,
 // decay the rows, M <- diag(a) M; correct what M holds for this key, e = beta (v - M^T k), M <- M + k e^T; read out y = M^T q.  q, k (kv_heads x dim) and v (heads x vdim) pass a
 // short causal convolution + SiLU; q, k are unit vectors per head; the decay and the output gate come from two-stage
-// (low-rank) projections whose inner sizes are the checkpoint's.
+// (low-rank) projections whose inner sizes are the checkpoint's.  head_decay: one decay per head, g = exp(-exp(A_log) softplus(W_a x + dt_bias)),
+// and full_gate: the output gate is silu(W_g x), both from one projection each.
 struct DeltaSpec {
 	int heads = 0, kv_heads = 0, dim = 0, vdim = 0, conv = 0;
+	bool head_decay = false, full_gate = false;
 	int decay_rank = 0, gate_rank = 0; // filled from the tensors' shapes at load
+	int conv_channels() const { return 2 * kv_heads * dim + heads * vdim; }
+};
+
+// Time mixing: each of five projections reads its own blend h + (h' - h) mu_s of the layer's input and the previous token's
+// (zero before the sequence); r, k, v per head; decay a = exp(-exp(W_2 tanh(W_1 x_w) + w_0)) per head and key channel.  Per head
+// y = (S + diag(u) k v^T)^T r with the stored bonus u, then S <- diag(a) S + k v^T; y is RMS-normed per head, times a weight per
+// channel, times silu(W_g x_g).
+struct WkvSpec {
+	int heads = 0, dim = 0;
+	int decay_rank = 0; // filled from the tensors' shapes at load
+	int inner() const { return heads * dim; }
 };
 
 struct FfnSpec {
@@ -149,6 +168,7 @@ struct LayerSpec {
 	DeltaSpec delta;
 	LatentSpec latent;
 	GlaSpec gla;
+	WkvSpec wkv;
 	float left_scale = 1.f, right_scale = 1.f; // Parallel: left_scale * attention + right_scale * delta rule
 	FfnSpec ffn;
 	// widths of what the layer computes per row, for scratch sizing
@@ -156,6 +176,20 @@ struct LayerSpec {
 	int mixed_width() const;   // the input of the output projection(s), summed over the mixers
 	int conv_width() const;    // channels that pass a short convolution
 	int aux_width() const;     // second-stage projections
+	int block_out_width() const { return mixed_width() + (ffn.kind == FfnSpec::Dense ? ffn.ff : 0); } // input of a packed block's one output product
+};
+
+// Bigram embedding: x += table[(previous token * mul_prev + token * mul_cur) mod buckets], the table's last row (number `buckets`)
+// for a sequence's first token.  The previous token is sequence state.
+struct BigramSpec {
+	int buckets = 0; // 0: none
+	long long mul_prev = 0, mul_cur = 0;
+};
+
+// One entry of the order in which the layers run.
+struct LayerRun {
+	int layer = 0;
+	bool add_embedding = false; // the embedding output is added to x right before this run
 };
 
 enum class TensorRole {
@@ -167,7 +201,9 @@ enum class TensorRole {
 	InConv1, InConv2, DepthWeights, RouterBias, SharedGate, SharedUp, SharedDown,
 	LatentDq, LatentDqNorm, LatentUq, LatentDkv, LatentDkvNorm, LatentUk, LatentUv,
 	GlaNorm, GlaDecay1, GlaDecay2, GlaDecayBias,
-	Norm1Post, Norm2Post, Sink, DiffLq1, DiffLk1, DiffLq2, DiffLk2, SideEmbed, SideGate, SideProj, SideNorm
+	Norm1Post, Norm2Post, Sink, DiffLq1, DiffLk1, DiffLq2, DiffLk2, SideEmbed, SideGate, SideProj, SideNorm,
+	Norm1Bias, FinalNormBias, Bigram, VBias, DeltaDecay, DeltaGate,
+	WkvR, WkvMuR, WkvMuK, WkvMuV, WkvMuG, WkvMuW, WkvDecay1, WkvDecay2, WkvDecayBias, WkvBonus, WkvNorm
 };
 
 struct StackSpec {
@@ -191,10 +227,18 @@ struct StackSpec {
 	bool sandwich_norm = false;    // a norm before and after every sublayer: x += norm_b(sublayer(norm_a(x)))
 	int token_side = 0;            // > 0: at the end of layer i, with e = the layer's slice [i token_side, (i + 1) token_side) of a second
 	                               // embedding of the token: y = P (gelu_tanh(G x) * e), x += y / sqrt(mean y^2 + eps) * w (plain weight)
+	bool norm_bias = false;        // layer norms add a stored bias
+	bool packed_block = false;     // with parallel_block: a dense feed-forward beside the mixer, run as one product in ([mixer's projections | gate | up]
+	                               // of the shared input) and one product out ([W_o | W_down] over [mixer output | activation])
+	BigramSpec bigram;
+	int loop_start = 0, loop_stop = 0, loop_times = 1; // layers loop_start .. loop_stop - 1 run loop_times times in a row with the same weights; every
+	                               // pass has its own caches and state, and the embedding output is added to x before every pass but the first
 	bool depth_average = false;    // what a layer hands on is a learned weighted sum of the embedding output and all layer results so far
 	// name of a tensor in the checkpoint; `expert` < 0 for tensors that are not per expert
 	std::string (*tensor_name)(int layer, TensorRole role, int expert) = nullptr;
 
+	std::vector<LayerRun> runs() const; // the layers in the order they run
+	int max_block_out() const;
 	int max_q_dim() const;  // max over layers of heads * dim
 	int max_kv_dim() const; // kv_heads * dim
 	int max_v_dim() const;  // kv_heads * vdim

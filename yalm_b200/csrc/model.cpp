@@ -105,6 +105,19 @@ size_t Config::active_bytes(size_t pos) const {
 		size_t total = 2 * W * ws + (size_t)s.vocab * W * ws + W * 4;
 		for (const yalm::LayerSpec &l : s.layers) {
 			const yalm::MixerSpec &m = l.mix;
+			if (s.packed_block) {
+				// per run of the layer: both products, norm weight and bias, then the mixer's own: the fp32 matrix state read and written, the
+				// convolution weights, the decay's second stage, or all earlier keys and values
+				const int i = (int)(&l - s.layers.data());
+				const size_t times = i >= s.loop_start && i < s.loop_stop ? s.loop_times : 1;
+				size_t b = ((size_t)l.proj_width() + l.block_out_width()) * W * ws + 2 * W * 4;
+				if (l.kind == yalm::MixerKind::DeltaRule) b += (size_t)2 * 4 * l.delta.heads * l.delta.dim * l.delta.vdim + (size_t)4 * l.delta.conv_channels() * 2 * l.delta.conv;
+				else if (l.kind == yalm::MixerKind::TimeMix)
+					b += (size_t)2 * 4 * l.wkv.inner() * l.wkv.dim + (size_t)l.wkv.inner() * l.wkv.decay_rank * ws + 6 * W * 4;
+				else b += (pos + 1) * m.kv_heads * (m.dim + m.vdim) * cb;
+				total += times * b;
+				continue;
+			}
 			if (s.parallel_block) {
 				// the packed projection and the output projection(s), the fp32 matrix state read and written, the window of keys
 				total += ((size_t)l.proj_width() + l.mixed_width()) * W * ws + 2 * W * 4;
@@ -865,7 +878,10 @@ int Model::launches_per_forward(InferenceMode mode) const {
 	if (config->stack) { // before any capture, the per-op route: embed + per layer: qkv, q/k norm + append, [pool], attention, wo, norm + residual, feed-forward (4) [+ final norm, head]
 		int n = 1;
 		for (const yalm::LayerSpec &l : config->stack->layers) {
-			if (config->stack->sandwich_norm) // norm, projection, mixer (latent 5 with the split merge, differential 4), output projection + norm; norm, up, activation, down + norm; side input
+			if (config->stack->packed_block) { // product in, mixer (1, attention 3 with the split merge), product out
+				const int i = (int)(&l - config->stack->layers.data());
+				n += (i >= config->stack->loop_start && i < config->stack->loop_stop ? config->stack->loop_times : 1) * (2 + (l.kind == yalm::MixerKind::Attention ? 3 : 1));
+			} else if (config->stack->sandwich_norm) // norm, projection, mixer (latent 5 with the split merge, differential 4), output projection + norm; norm, up, activation, down + norm; side input
 				n += 2 + (l.kind == yalm::MixerKind::LatentAttention ? 5 : 4) + 1 + (l.ffn.kind == yalm::FfnSpec::None ? 0 : 4) + (config->stack->token_side > 0 ? 1 : 0);
 			else if (config->stack->parallel_block) // norm + shift, projection, mixer (state space 5, parallel 14), experts 3, residual
 				n += 3 + (l.kind == yalm::MixerKind::StateSpace ? 5 : 14) + (l.ffn.kind == yalm::FfnSpec::None ? 0 : 3);

@@ -5,6 +5,7 @@
 //
 // Mechanisms (each with its constants as parameters, so another layered design can use them):
 //   embed_rows            x = E[token] (+ learned position row)
+//   embed_bigram_rows     x = E[token] + B[hash of the previous token and this one]
 //   linear_rows           y = alpha * x W^T: warp-per-output GEMV for few rows, 64 x 64 SIMT tiles for many (the tensor-core
 //                         route for 16-bit weights is prefill_gemm.cu; this is the exact-fp32 and odd-shape route)
 //   qkv_post_rows         RMS norm over the whole q / k projection, value blending with an earlier layer's values, append
@@ -41,6 +42,33 @@ __global__ void embed_rows_kernel(float *__restrict__ x, const void *__restrict_
 		float v = Elem<DT>::get(table, (size_t)tok * dim + e) * scale;
 		if (positions) v += Elem<DT>::get(positions, (size_t)p * dim + e);
 		x[(size_t)m * dim + e] = v;
+	}
+}
+
+// x = E[token] + B[row], row = (previous token * mul_prev + token * mul_cur) mod buckets, the last row (number `buckets`) at
+// position 0; also to x0 (optional).  The previous token of the call's first row is `prev` (device word), which then takes the
+// last row's token: in this kernel for one-row calls (its only CTA has read it), by the launcher otherwise.
+template <int DT>
+__global__ void embed_bigram_rows_kernel(float *__restrict__ x, float *__restrict__ x0, const void *__restrict__ table, const void *__restrict__ bigram,
+                                         const int *__restrict__ tokens, int buckets, long long mul_prev, long long mul_cur, int *prev, int dim, int pos0,
+                                         const int *__restrict__ ctl) {
+	const int m = blockIdx.x;
+	const int tok = tokens ? tokens[m] : ctl[CTL_TOKEN];
+	const int p = first_pos(ctl, pos0) + m;
+	long long row = buckets;
+	if (p > 0) {
+		const int before = m > 0 ? tokens[m - 1] : *prev;
+		row = ((long long)before * mul_prev + (long long)tok * mul_cur) % buckets;
+		if (row < 0) row += buckets;
+	}
+	for (int e = threadIdx.x; e < dim; e += blockDim.x) {
+		const float v = Elem<DT>::get(table, (size_t)tok * dim + e) + Elem<DT>::get(bigram, (size_t)row * dim + e);
+		x[(size_t)m * dim + e] = v;
+		if (x0) x0[(size_t)m * dim + e] = v;
+	}
+	if (gridDim.x == 1) {
+		__syncthreads();
+		if (threadIdx.x == 0) *prev = tok;
 	}
 }
 
@@ -774,6 +802,15 @@ extern "C" int yalm_embed_rows(float *x, const void *table, const void *position
                                const int *ctl, float scale, yalm_stream_t s) {
 	if (!x || !table || n < 1 || dim < 1 || (!tokens && !ctl)) return YALM_EINVAL;
 	DISPATCH_DT(dtype, (embed_rows_kernel<DT><<<n, 256, 0, (cudaStream_t)s>>>(x, table, positions, tokens, dim, pos0, ctl, scale)));
+	return (int)cudaGetLastError();
+}
+
+extern "C" int yalm_embed_bigram_rows(float *x, float *x0, const void *table, const void *bigram, int dtype, const int *tokens, int buckets, long long mul_prev,
+                                      long long mul_cur, int *prev, int n, int dim, int pos0, const int *ctl, yalm_stream_t s) {
+	if (!x || !table || !bigram || !prev || buckets < 1 || n < 1 || dim < 1 || (!tokens && (!ctl || n > 1))) return YALM_EINVAL;
+	cudaStream_t st = (cudaStream_t)s;
+	DISPATCH_DT(dtype, (embed_bigram_rows_kernel<DT><<<n, 256, 0, st>>>(x, x0, table, bigram, tokens, buckets, mul_prev, mul_cur, prev, dim, pos0, ctl)));
+	if (n > 1) return (int)cudaMemcpyAsync(prev, tokens + n - 1, sizeof(int), cudaMemcpyDeviceToDevice, st);
 	return (int)cudaGetLastError();
 }
 

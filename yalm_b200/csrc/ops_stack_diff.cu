@@ -14,7 +14,9 @@ namespace stack {
 // Row m of the packed projection P (ld): nqv query vectors of dk channels from o_q, nkv key vectors from o_k, nvh value heads
 // of dv channels from o_v.  Every query and key vector: RMS norm over its dk channels with the shared weight qw / kw (null:
 // none), then its first rot_dims channels turned by the row's position (pair i = channels (i, i + rot_dims / 2), or
-// (2 i, 2 i + 1) if interleaved).  Queries stay in place; key vector j goes to kring (j, slot, channel), value head j to vring;
+// (2 i, 2 i + 1) if interleaved).  Biases qb / kb / vb (one per channel of all vectors; null: none) are added first; norm_after
+// != 0: every vector is divided by its root mean square after the rotation, without a weight, instead of the norm before it.
+// Queries stay in place; key vector j goes to kring (j, slot, channel), value head j to vring;
 // positions below `keep` also go, as the ring holds them, to kfirst (j, keep, dk) / vfirst (j, keep, dv) in fp32, from where
 // the attention reads the tokens that stay visible after they have left the window.  A warp owns a vector.
 constexpr int kHnWarps = 8, kHnMaxDim = 512;
@@ -25,7 +27,8 @@ __global__ void __launch_bounds__(kHnWarps * 32) head_norm_rope_append_rows_kern
                                                                                   int rot_dims, int interleaved, float eps, CT *__restrict__ kring,
                                                                                   CT *__restrict__ vring, int ring, float *__restrict__ kfirst,
                                                                                   float *__restrict__ vfirst, int keep, int pos0,
-                                                                                  const int *__restrict__ ctl) {
+                                                                                  const int *__restrict__ ctl, const float *__restrict__ qb,
+                                                                                  const float *__restrict__ kb, const float *__restrict__ vb, int norm_after) {
 	__shared__ float buf[kHnWarps][kHnMaxDim];
 	const int m = blockIdx.x, p = first_pos(ctl, pos0) + m, slot = p % ring;
 	const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, half = rot_dims / 2;
@@ -33,10 +36,10 @@ __global__ void __launch_bounds__(kHnWarps * 32) head_norm_rope_append_rows_kern
 	for (int v = blockIdx.y * kHnWarps + warp; v < nqv + nkv; v += gridDim.y * kHnWarps) { // grid.y spreads a row's vectors over CTAs
 		const bool is_q = v < nqv;
 		float *src = row + (is_q ? o_q + (size_t)v * dk : o_k + (size_t)(v - nqv) * dk);
-		const float *w = is_q ? qw : kw;
+		const float *w = is_q ? qw : kw, *bias = is_q ? (qb ? qb + (size_t)v * dk : nullptr) : (kb ? kb + (size_t)(v - nqv) * dk : nullptr);
 		float ss = 0.f;
 		for (int d = lane; d < dk; d += 32) {
-			const float x = src[d];
+			const float x = src[d] + (bias ? bias[d] : 0.f);
 			vs[d] = x, ss += x * x;
 		}
 		ss = warp_sum(ss);
@@ -46,7 +49,7 @@ __global__ void __launch_bounds__(kHnWarps * 32) head_norm_rope_append_rows_kern
 		__syncwarp();
 		CT *kdst = is_q ? nullptr : kring + ((size_t)(v - nqv) * ring + slot) * dk;
 		float *fdst = (!is_q && p < keep) ? kfirst + ((size_t)(v - nqv) * keep + p) * dk : nullptr;
-		for (int d = lane; d < dk; d += 32) {
+		auto turned = [&](int d) {
 			float o = vs[d];
 			if (d < rot_dims) {
 				const int i = interleaved ? d >> 1 : (d < half ? d : d - half);
@@ -57,6 +60,35 @@ __global__ void __launch_bounds__(kHnWarps * 32) head_norm_rope_append_rows_kern
 				sn *= mag, cs *= mag;
 				o = first ? a * cs - b * sn : b * cs + a * sn;
 			}
+			return o;
+		};
+		if (norm_after) { // the vector's rotated channels stay in this lane's registers while their mean square is formed
+			constexpr int N = kHnMaxDim / 32;
+			float ov[N], s2 = 0.f;
+#pragma unroll
+			for (int j = 0; j < N; ++j) {
+				if (j * 32 >= dk) break;
+				const int d = j * 32 + lane;
+				ov[j] = d < dk ? turned(d) : 0.f;
+				s2 += ov[j] * ov[j];
+			}
+			const float rr = 1.0f / sqrtf(warp_sum(s2) / (float)dk + eps);
+#pragma unroll
+			for (int j = 0; j < N; ++j) {
+				if (j * 32 >= dk) break;
+				const int d = j * 32 + lane;
+				if (d >= dk) continue;
+				if (is_q) src[d] = ov[j] * rr;
+				else {
+					cache_put(kdst, d, ov[j] * rr);
+					if (fdst) fdst[d] = cache_get(kdst, d);
+				}
+			}
+			__syncwarp();
+			continue;
+		}
+		for (int d = lane; d < dk; d += 32) {
+			const float o = turned(d);
 			if (is_q) src[d] = o;
 			else {
 				cache_put(kdst, d, o);
@@ -68,7 +100,7 @@ __global__ void __launch_bounds__(kHnWarps * 32) head_norm_rope_append_rows_kern
 	for (int e = blockIdx.y * blockDim.x + threadIdx.x; e < nvh * dv; e += gridDim.y * blockDim.x) {
 		const int g = e / dv, d = e % dv;
 		CT *dst = vring + ((size_t)g * ring + slot) * dv;
-		cache_put(dst, d, row[o_v + e]);
+		cache_put(dst, d, row[o_v + e] + (vb ? vb[e] : 0.f));
 		if (p < keep) vfirst[((size_t)g * keep + p) * dv + d] = cache_get(dst, d);
 	}
 }
@@ -162,26 +194,42 @@ __global__ void token_side_act_rows_kernel(float *__restrict__ h, int ldh, const
 using namespace yalm;
 using namespace yalm::stack;
 
-extern "C" int yalm_head_norm_rope_append_rows(float *proj, int ld, int o_q, int o_k, int o_v, int n_q_vectors, int n_k_vectors, int n_v_heads, int dk, int dv,
-                                               const float *q_norm, const float *k_norm, const float *freq, float magnitude, int rot_dims, int interleaved,
-                                               float eps, void *key_ring, void *value_ring, int ring, float *key_first, float *value_first, int keep,
-                                               int cache_f32, int n, int pos0, const int *ctl, yalm_stream_t s) {
+static int head_append(float *proj, int ld, int o_q, int o_k, int o_v, int n_q_vectors, int n_k_vectors, int n_v_heads, int dk, int dv, const float *q_norm,
+                       const float *k_norm, const float *freq, float magnitude, int rot_dims, int interleaved, float eps, void *key_ring, void *value_ring,
+                       int ring, float *key_first, float *value_first, int keep, int cache_f32, int n, int pos0, const int *ctl, const float *q_bias,
+                       const float *k_bias, const float *v_bias, int norm_after, cudaStream_t st) {
 	if (!proj || !key_ring || !value_ring || n < 1 || ring < 1 || dk < 1 || dk > kHnMaxDim || dv < 1 || rot_dims < 0 || rot_dims > dk || rot_dims % 2 ||
 	    (rot_dims > 0 && !freq) || keep < 0 || (keep > 0 && (!key_first || !value_first)))
 		return YALM_EINVAL;
-	cudaStream_t st = (cudaStream_t)s;
 	// every load of a vector's chain (channels, norm, rotation, store) waits for the one before it: enough warps in flight hide that
 	const dim3 grid(n, std::max(1, std::min((n_q_vectors + n_k_vectors + kHnWarps - 1) / kHnWarps, n >= 64 ? 4 : 16)));
 	if (cache_f32)
 		head_norm_rope_append_rows_kernel<float><<<grid, kHnWarps * 32, 0, st>>>(proj, ld, o_q, o_k, o_v, n_q_vectors, n_k_vectors, n_v_heads, dk, dv, q_norm, k_norm,
 		                                                                       freq, magnitude, rot_dims, interleaved, eps, (float *)key_ring, (float *)value_ring,
-		                                                                       ring, key_first, value_first, keep, pos0, ctl);
+		                                                                       ring, key_first, value_first, keep, pos0, ctl, q_bias, k_bias, v_bias, norm_after);
 	else
 		head_norm_rope_append_rows_kernel<__nv_bfloat16><<<grid, kHnWarps * 32, 0, st>>>(proj, ld, o_q, o_k, o_v, n_q_vectors, n_k_vectors, n_v_heads, dk, dv, q_norm,
 		                                                                               k_norm, freq, magnitude, rot_dims, interleaved, eps,
 		                                                                               (__nv_bfloat16 *)key_ring, (__nv_bfloat16 *)value_ring, ring, key_first,
-		                                                                               value_first, keep, pos0, ctl);
+		                                                                               value_first, keep, pos0, ctl, q_bias, k_bias, v_bias, norm_after);
 	return (int)cudaGetLastError();
+}
+
+extern "C" int yalm_head_norm_rope_append_rows(float *proj, int ld, int o_q, int o_k, int o_v, int n_q_vectors, int n_k_vectors, int n_v_heads, int dk, int dv,
+                                               const float *q_norm, const float *k_norm, const float *freq, float magnitude, int rot_dims, int interleaved,
+                                               float eps, void *key_ring, void *value_ring, int ring, float *key_first, float *value_first, int keep,
+                                               int cache_f32, int n, int pos0, const int *ctl, yalm_stream_t s) {
+	return head_append(proj, ld, o_q, o_k, o_v, n_q_vectors, n_k_vectors, n_v_heads, dk, dv, q_norm, k_norm, freq, magnitude, rot_dims, interleaved, eps, key_ring,
+	                   value_ring, ring, key_first, value_first, keep, cache_f32, n, pos0, ctl, nullptr, nullptr, nullptr, 0, (cudaStream_t)s);
+}
+
+// Biases first (each null: none), then the rotation, then every query / key vector divided by its root mean square (no weight).
+extern "C" int yalm_head_bias_rope_norm_append_rows(float *proj, int ld, int o_q, int o_k, int o_v, int n_q_vectors, int n_k_vectors, int n_v_heads, int dk,
+                                                    int dv, const float *q_bias, const float *k_bias, const float *v_bias, const float *freq, float magnitude,
+                                                    int rot_dims, int interleaved, float eps, void *key_ring, void *value_ring, int ring, int cache_f32, int n,
+                                                    int pos0, const int *ctl, yalm_stream_t s) {
+	return head_append(proj, ld, o_q, o_k, o_v, n_q_vectors, n_k_vectors, n_v_heads, dk, dv, nullptr, nullptr, freq, magnitude, rot_dims, interleaved, eps, key_ring,
+	                   value_ring, ring, nullptr, nullptr, 0, cache_f32, n, pos0, ctl, q_bias, k_bias, v_bias, 1, (cudaStream_t)s);
 }
 
 extern "C" int yalm_diff_combine_rows(float *out, int ldo, const float *maps, int ldm, const float *gate, int ldg, int n, int heads, int dv, float lambda,

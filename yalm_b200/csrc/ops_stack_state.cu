@@ -11,6 +11,8 @@
 //   conv_act_rows          per-channel causal convolution over the last `taps` positions (+ bias) and SiLU
 //   state_scan_rows        M <- a * M;  e = beta (v - M^T k)  or  e = vscale * v;  M <- M + k e^T;  y = M^T q (+ skip * v)
 //                          with a scalar or per-key-channel decay: both the state-space recurrence and the gated delta rule
+//   state_scan_bonus_rows  y = (M + diag(u) k v^T)^T q, then M <- a * M + k v^T: the read-out comes before the decay, with a bonus u per
+//                          head and key channel for the current position (time mixing)
 //   ssm_prep_rows          dt = softplus(raw + bias), decay = exp(-exp(A_log) dt)
 //   delta_prep_rows        unit q / k per head, beta = sigmoid(raw), per-channel decay from raw step sizes
 //   gated_group_norm_rows  rms over equal parts of (y * silu(z)), times a weight
@@ -124,6 +126,7 @@ struct ScanArgs {
 	int n, H, rep, D, P, pos0;
 	const int *ctl;
 	int vec; // k, q and per-channel decay rows are 16-byte aligned: 16-byte copies
+	const float *bonus = nullptr; // (H, D)
 };
 constexpr int kScanCols = 16, kScanTok = 8, kScanMaxD = 256;
 
@@ -157,7 +160,7 @@ __device__ __forceinline__ void load_seg(float (&r)[EPL], const float *p) {
 		r[0] = p[0];
 }
 
-template <int EPL>
+template <int EPL, bool BONUS>
 __global__ void __launch_bounds__(kScanCols * 8) state_scan_kernel(ScanArgs a) {
 	using LO = ScanLayout<EPL>;
 	constexpr int SEG = LO::SEG, DP = LO::DP, TOK = kScanTok, STAGE = LO::STAGE;
@@ -171,6 +174,10 @@ __global__ void __launch_bounds__(kScanCols * 8) state_scan_kernel(ScanArgs a) {
 #pragma unroll
 	for (int e = 0; e < EPL; ++e) s[e] = (!fresh && sub * EPL + e < a.D) ? sp[e] : 0.f;
 	const float skip = a.skip ? a.skip[h] : 0.f;
+	float bu[BONUS ? EPL : 1];
+	if constexpr (BONUS)
+#pragma unroll
+		for (int e = 0; e < EPL; ++e) bu[e] = sub * EPL + e < a.D ? a.bonus[(size_t)h * a.D + sub * EPL + e] : 0.f;
 	// what the copies never write: rows past D, the padding, columns past P, and the defaults of absent per-position scalars
 	for (int idx = tid; idx < 2 * STAGE; idx += blockDim.x) {
 		const int r = idx % STAGE;
@@ -224,6 +231,22 @@ __global__ void __launch_bounds__(kScanCols * 8) state_scan_kernel(ScanArgs a) {
 			load_seg<EPL>(kt, ks + t * DP + sub * SEG);
 			load_seg<EPL>(qt, qs + t * DP + sub * SEG);
 			const float vv = vs[t * kScanCols + col];
+			if constexpr (BONUS) { // read-out of the state as it was, then decay and update
+				float gt[EPL];
+				load_seg<EPL>(gt, gs + t * DP + sub * SEG);
+				po += __shfl_xor_sync(kFull, po, 4), po += __shfl_xor_sync(kFull, po, 2), po += __shfl_xor_sync(kFull, po, 1);
+				if (pout && sub == 0 && live) *pout = po;
+				float o4[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+				for (int e = 0; e < EPL; ++e) {
+					const float kv = kt[e] * vv;
+					o4[e & 3] = fmaf(fmaf(bu[e], kv, s[e]), qt[e], o4[e & 3]);
+					s[e] = fmaf(gt[e], s[e], kv);
+				}
+				po = (o4[0] + o4[1]) + (o4[2] + o4[3]);
+				pout = a.out + (size_t)(t0 + t) * a.ldo + h * a.P + min(c0 + col, a.P - 1);
+				continue;
+			}
 			if (a.decay_per_channel) {
 				float gt[EPL];
 				load_seg<EPL>(gt, gs + t * DP + sub * SEG);
@@ -633,6 +656,28 @@ extern "C" int yalm_conv_act_rows(float *out, int ldo, const float *in, int ldi,
 	return (int)cudaGetLastError();
 }
 
+template <bool BONUS>
+static int launch_scan(const ScanArgs &a, dim3 grid, cudaStream_t st) {
+#define SCAN_CASE(EPL_)                                                                                                                      \
+	{                                                                                                                                        \
+		constexpr size_t smem = sizeof(float) * 2 * ScanLayout<EPL_>::STAGE;                                                                 \
+		static bool configured = false;                                                                                                      \
+		if (smem > 48 * 1024 && !configured) {                                                                                               \
+			YALM_TRY(cudaFuncSetAttribute(state_scan_kernel<EPL_, BONUS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));          \
+			configured = true;                                                                                                               \
+		}                                                                                                                                    \
+		state_scan_kernel<EPL_, BONUS><<<grid, kScanCols * 8, smem, st>>>(a);                                                                \
+	}
+	if (a.D <= 8) SCAN_CASE(1)
+	else if (a.D <= 16) SCAN_CASE(2)
+	else if (a.D <= 32) SCAN_CASE(4)
+	else if (a.D <= 64) SCAN_CASE(8)
+	else if (a.D <= 128) SCAN_CASE(16)
+	else SCAN_CASE(32)
+#undef SCAN_CASE
+	return (int)cudaGetLastError();
+}
+
 // See ScanArgs.  k, q: (n, kv heads * D) with head h reading kv head h / rep; v, out: (n, H * P); decay: (n, H) or, with
 // decay_per_channel, (n, H * D); vscale, beta: (n, H) or null; skip: (H) or null; state: (H, P, D) fp32.  D <= 256.
 extern "C" int yalm_state_scan_rows(float *out, int ldo, const float *k, int ldk, const float *q, int ldq, const float *v, int ldv, const float *decay,
@@ -643,25 +688,17 @@ extern "C" int yalm_state_scan_rows(float *out, int ldo, const float *k, int ldk
 	const int vec = D % 4 == 0 && al(k, ldk) && al(q, ldq) && (!decay_per_channel || al(decay, ldd));
 	ScanArgs a{out, ldo, k, q, v, decay, vscale, beta, skip, ldk, ldq, ldv, ldd, ldvs, ldb, decay_per_channel, state, n, heads, rep, D, P, pos0, ctl, vec};
 	const dim3 grid((P + kScanCols - 1) / kScanCols, heads);
-	cudaStream_t st = (cudaStream_t)s;
-#define SCAN_CASE(EPL_)                                                                                                                      \
-	{                                                                                                                                        \
-		constexpr size_t smem = sizeof(float) * 2 * ScanLayout<EPL_>::STAGE;                                                                 \
-		static bool configured = false;                                                                                                      \
-		if (smem > 48 * 1024 && !configured) {                                                                                               \
-			YALM_TRY(cudaFuncSetAttribute(state_scan_kernel<EPL_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));                 \
-			configured = true;                                                                                                               \
-		}                                                                                                                                    \
-		state_scan_kernel<EPL_><<<grid, kScanCols * 8, smem, st>>>(a);                                                                       \
-	}
-	if (D <= 8) SCAN_CASE(1)
-	else if (D <= 16) SCAN_CASE(2)
-	else if (D <= 32) SCAN_CASE(4)
-	else if (D <= 64) SCAN_CASE(8)
-	else if (D <= 128) SCAN_CASE(16)
-	else SCAN_CASE(32)
-#undef SCAN_CASE
-	return (int)cudaGetLastError();
+	return launch_scan<false>(a, grid, (cudaStream_t)s);
+}
+
+// The time-mixing recurrence: out = (M + diag(bonus) k v^T)^T q, M <- decay M + k v^T; k, q, decay (n, H D), v, out (n, H P), bonus (H, D).
+extern "C" int yalm_state_scan_bonus_rows(float *out, int ldo, const float *k, int ldk, const float *q, int ldq, const float *v, int ldv, const float *decay,
+                                          int ldd, const float *bonus, float *state, int n, int heads, int D, int P, int pos0, const int *ctl, yalm_stream_t s) {
+	if (!out || !k || !q || !v || !decay || !bonus || !state || n < 1 || heads < 1 || D < 1 || D > kScanMaxD || P < 1) return YALM_EINVAL;
+	auto al = [](const float *p, int ld) { return ((uintptr_t)p & 15) == 0 && ld % 4 == 0; };
+	ScanArgs a{out, ldo, k, q, v, decay, nullptr, nullptr, nullptr, ldk, ldq, ldv, ldd, 0, 0, 1, state, n, heads, 1, D, P, pos0, ctl,
+	           D % 4 == 0 && al(k, ldk) && al(q, ldq) && al(decay, ldd), bonus};
+	return launch_scan<true>(a, dim3((P + kScanCols - 1) / kScanCols, heads), (cudaStream_t)s);
 }
 
 extern "C" int yalm_ssm_prep_rows(float *dt, int lddt, float *decay, int ldd, const float *dt_bias, const float *a_log, int n, int heads, yalm_stream_t s) {

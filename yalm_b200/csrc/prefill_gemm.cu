@@ -41,6 +41,8 @@ struct GemmArgs {
 	int ldc;
 	float alpha; // kStoreF32 / kAddF32: the product is scaled before it is stored / added
 	int bf16;    // operands are bf16 instead of fp16 (same instruction kind, other format bits and tensor-map type)
+	int nseg;    // > 0: output columns [seg_end[s - 1], seg_end[s]) multiply rows s M .. s M + M - 1 of A (one input per segment)
+	int seg_end[8];
 };
 
 // ---- PTX ---------------------------------------------------------------------------------------------------------
@@ -130,7 +132,17 @@ gemm_f16_kernel(const __grid_constant__ CUtensorMap ta, const __grid_constant__ 
 	const uint32_t bars = base + kStages * kStage;           // full[kStages] | empty[kStages] | accumulator ready | TMEM address
 	const uint32_t full0 = bars, empty0 = bars + 8 * kStages, acc_bar = bars + 16 * kStages, tslot = acc_bar + 8;
 	const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-	const int m0 = blockIdx.x * BM, n0 = blockIdx.y * BN;
+	const int m0 = blockIdx.x * BM;
+	int n0 = blockIdx.y * BN, a0 = m0, n_end = g.N;
+	if (g.nseg > 0) { // tiles never straddle two segments
+		int t = blockIdx.y, start = 0, s = 0;
+		for (; s < g.nseg - 1; ++s) {
+			const int tiles = (g.seg_end[s] - start + BN - 1) / BN;
+			if (t < tiles) break;
+			t -= tiles, start = g.seg_end[s];
+		}
+		n0 = start + t * BN, n_end = g.seg_end[s], a0 = s * g.M + m0;
+	}
 	const int nkb = (g.K + BK - 1) / BK;
 
 	if (threadIdx.x == 0) {
@@ -152,7 +164,7 @@ gemm_f16_kernel(const __grid_constant__ CUtensorMap ta, const __grid_constant__ 
 				if (r > 0) mbar_wait(empty0 + 8 * s, (uint32_t)(r - 1) & 1u);
 				const uint32_t dst = base + s * kStage, bar = full0 + 8 * s;
 				mbar_expect_tx(bar, kStage);
-				tma_load_2d(dst, &ta, kb * BK, m0, bar);
+				tma_load_2d(dst, &ta, kb * BK, a0, bar);
 				tma_load_2d(dst + kTileBytes, &tb, kb * BK, n0, bar);
 				if (NB == 2) tma_load_2d(dst + 2 * kTileBytes, &tb2, kb * BK, n0, bar);
 			}
@@ -193,7 +205,7 @@ gemm_f16_kernel(const __grid_constant__ CUtensorMap ta, const __grid_constant__ 
 					__half *dst = g.h + (size_t)row * g.ldc + col;
 #pragma unroll
 					for (int i = 0; i < 32; i += 8) {
-						if (col + i + 8 <= g.N) {
+						if (col + i + 8 <= n_end) {
 							uint4 pk;
 							__half2 h0 = __floats2half2_rn(v[i], v[i + 1]), h1 = __floats2half2_rn(v[i + 2], v[i + 3]);
 							__half2 h2 = __floats2half2_rn(v[i + 4], v[i + 5]), h3 = __floats2half2_rn(v[i + 6], v[i + 7]);
@@ -201,14 +213,14 @@ gemm_f16_kernel(const __grid_constant__ CUtensorMap ta, const __grid_constant__ 
 							pk.z = *reinterpret_cast<uint32_t *>(&h2), pk.w = *reinterpret_cast<uint32_t *>(&h3);
 							*reinterpret_cast<uint4 *>(dst + i) = pk;
 						} else {
-							for (int j = i; j < i + 8 && col + j < g.N; ++j) dst[j] = __float2half_rn(v[j]);
+							for (int j = i; j < i + 8 && col + j < n_end; ++j) dst[j] = __float2half_rn(v[j]);
 						}
 					}
 				} else {
 					float *dst = g.c + (size_t)row * g.ldc + col;
 #pragma unroll
 					for (int i = 0; i < 32; i += 4) {
-						if (col + i + 4 <= g.N) {
+						if (col + i + 4 <= n_end) {
 							float4 o = make_float4(g.alpha * v[i], g.alpha * v[i + 1], g.alpha * v[i + 2], g.alpha * v[i + 3]);
 							if (g.tail == kAddF32) { // x += W v (src/infer.cpp:335-337), residual stream stays fp32
 								const float4 x = *reinterpret_cast<const float4 *>(dst + i);
@@ -216,7 +228,7 @@ gemm_f16_kernel(const __grid_constant__ CUtensorMap ta, const __grid_constant__ 
 							}
 							*reinterpret_cast<float4 *>(dst + i) = o;
 						} else {
-							for (int j = i; j < i + 4 && col + j < g.N; ++j) dst[j] = g.tail == kAddF32 ? dst[j] + g.alpha * v[j] : g.alpha * v[j];
+							for (int j = i; j < i + 4 && col + j < n_end; ++j) dst[j] = g.tail == kAddF32 ? dst[j] + g.alpha * v[j] : g.alpha * v[j];
 						}
 					}
 				}
@@ -270,7 +282,12 @@ static int launch(const CUtensorMap &ta, const CUtensorMap &tb, const CUtensorMa
 		YALM_TRY(cudaFuncSetAttribute(gemm_f16_kernel<NB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
 		configured = true;
 	}
-	const dim3 grid((g.M + BM - 1) / BM, (g.N + BN - 1) / BN);
+	int ntiles = (g.N + BN - 1) / BN;
+	if (g.nseg > 0) {
+		ntiles = 0;
+		for (int i = 0, at = 0; i < g.nseg; ++i) ntiles += (g.seg_end[i] - at + BN - 1) / BN, at = g.seg_end[i];
+	}
+	const dim3 grid((g.M + BM - 1) / BM, ntiles);
 	gemm_f16_kernel<NB><<<grid, kGemmThreads, smem, st>>>(ta, tb, tb2, g);
 	return (int)cudaGetLastError();
 }
@@ -289,7 +306,25 @@ extern "C" int yalm_gemm_16(float *c, int ldc, const void *a, const void *w, int
 	int rc = make_map(&ta, a, M, K, bf16 != 0);
 	if (!rc) rc = make_map(&tb, w, N, K, bf16 != 0);
 	if (rc) return rc;
-	GemmArgs g{M, N, K, accumulate ? kAddF32 : kStoreF32, 0, c, nullptr, ldc, alpha, bf16 != 0};
+	GemmArgs g{M, N, K, accumulate ? kAddF32 : kStoreF32, 0, c, nullptr, ldc, alpha, bf16 != 0, 0, {}};
+	return launch<1>(ta, tb, tb, g, (cudaStream_t)s);
+}
+// The same with one input per segment of output columns: columns [segment_end[i - 1], segment_end[i]) of c = a_i w^T, a_i = rows
+// i M .. i M + M - 1 of a (n_segments M, K).  Segment bounds are multiples of 4 (the last one is N).
+extern "C" int yalm_gemm_16_segments(float *c, int ldc, const void *a, const void *w, int M, int N, int K, int n_segments, const int *segment_end, int bf16,
+                                     yalm_stream_t s) {
+	if (!c || !a || !w || M < 1 || N < 1 || K < 8 || K % 8 || ldc < N || ldc % 4 || ((uintptr_t)a & 15) || ((uintptr_t)w & 15) || ((uintptr_t)c & 15) || n_segments < 1 ||
+	    n_segments > 8 || !segment_end || segment_end[n_segments - 1] != N)
+		return YALM_EINVAL;
+	GemmArgs g{M, N, K, kStoreF32, 0, c, nullptr, ldc, 1.0f, bf16 != 0, n_segments, {}};
+	for (int i = 0, at = 0; i < n_segments; ++i) {
+		if (segment_end[i] <= at || (i + 1 < n_segments && segment_end[i] % 4)) return YALM_EINVAL;
+		g.seg_end[i] = at = segment_end[i];
+	}
+	CUtensorMap ta, tb;
+	int rc = make_map(&ta, a, n_segments * M, K, bf16 != 0);
+	if (!rc) rc = make_map(&tb, w, N, K, bf16 != 0);
+	if (rc) return rc;
 	return launch<1>(ta, tb, tb, g, (cudaStream_t)s);
 }
 extern "C" int yalm_gemm_f16(float *c, int ldc, const void *a, const void *w, int M, int N, int K, int accumulate, yalm_stream_t s) {
@@ -305,7 +340,7 @@ extern "C" int yalm_gemm_glu_f16(void *h, int ldh, const void *a, const void *w1
 	if (!rc) rc = make_map(&tb, w1, N, K);
 	if (!rc) rc = make_map(&tb2, w3, N, K);
 	if (rc) return rc;
-	GemmArgs g{M, N, K, kGluF16, act, nullptr, static_cast<__half *>(h), ldh, 1.0f, 0};
+	GemmArgs g{M, N, K, kGluF16, act, nullptr, static_cast<__half *>(h), ldh, 1.0f, 0, 0, {}};
 	return launch<2>(ta, tb, tb2, g, (cudaStream_t)s);
 }
 

@@ -98,6 +98,15 @@ struct StackLayer {
 	// differential attention: columns [q: map, head | k: map, kv head | v | one gate number per head]; kring holds maps * kv heads key
 	// vectors per slot, vring kv heads; kpool / vpool (max_blocks = keep_first entries) the window's kept first tokens
 	float lambda = 0.f;
+	// ---- parallel blocks with one product in and one out: wproj is [mixer | gate | up | rest], wout [W_o | W_down] row by row ----
+	float *norm1_bias = nullptr;
+	int o_glu = 0;                                            // gate rows, then up rows
+	float *mu = nullptr;                                      // time mixing: one blend weight row per output segment (zero rows for plain ones)
+	float *bonus = nullptr;                                   // (heads, dim)
+	std::vector<int> seg_end;                                 // output columns of every segment of wproj
+	int plain_mask = 0;                                       // segments that read the norm's output itself
+	bool add_embedding = false;                               // the embedding output is added to x right before this layer run
+	const StackLayer *shares = nullptr;                       // a repeated pass of that layer: its weights, own caches and state
 	void *side_gate = nullptr, *side_proj = nullptr;          // token side input: (token_side, dim), (dim, token_side)
 	float *side_norm = nullptr;
 };
@@ -142,6 +151,10 @@ int Config::from_json(YALMData &data, int context, int compute) {
 			}
 		}
 		if (l.kind == yalm::MixerKind::LinearAttention && (l.gla.decay_rank = rows(TensorRole::GlaDecay1)) < 1) {
+			fprintf(stderr, "yalm_b200: layer %d: the decay's two-stage projection is missing\n", i);
+			return YALM_EFORMAT;
+		}
+		if (l.kind == yalm::MixerKind::TimeMix && (l.wkv.decay_rank = rows(TensorRole::WkvDecay1)) < 1) {
 			fprintf(stderr, "yalm_b200: layer %d: the decay's two-stage projection is missing\n", i);
 			return YALM_EFORMAT;
 		}
@@ -251,6 +264,9 @@ struct Model::StackScratch {
 	      *logits = nullptr, *probs = nullptr;
 	void *a16 = nullptr, *a16e = nullptr, *a16r = nullptr; // 16-bit operands of the tensor-core products: main stream, experts' stream, second mixer's stream
 	float *hs = nullptr, *conv = nullptr, *aux = nullptr, *scan = nullptr, *att2 = nullptr, *y1 = nullptr, *y2 = nullptr; // parallel blocks
+	float *mix = nullptr, *blk = nullptr, *x0 = nullptr; // packed blocks: the blends, the output product's input; the embedding output (repeated passes)
+	int *prev = nullptr;      // bigram embedding: the previous position's token (sequence state)
+	bool x0_added = false;    // x already holds the embedding output the next layer run asks for (added by the previous product's epilogue)
 	float *hsh = nullptr;     // the shared expert's hidden rows (the routed experts' are in h)
 	float *hist = nullptr;    // weighted sum over depth: the embedding output and every layer's result of the current rows, (layers + 1, cap, width)
 	void *lat16 = nullptr, *lat_ek = nullptr, *lat_ev = nullptr; // latent attention, prompt portions: latents of the visible rows (bf16), keys / values per head
@@ -303,6 +319,8 @@ void Model::build_stack(YALMData &data) {
 	if (s.learned_positions) pl.push_back({&_pos_table, {mat(tensor(0, TensorRole::Positions, -1, {s.max_positions, s.width}))}});
 	pl.push_back({(void **)&rms_final_weight, {vec32(s.norm_scalar ? tensor(0, TensorRole::FinalNorm, -1, {}) : tensor(0, TensorRole::FinalNorm, -1, {s.width}))}});
 	if (s.token_side > 0) pl.push_back({&_side_table, {mat(tensor(0, TensorRole::SideEmbed, -1, {s.vocab, s.token_side * (int)s.layers.size()}))}});
+	if (s.norm_bias) pl.push_back({(void **)&_final_bias, {vec32(tensor(0, TensorRole::FinalNormBias, -1, {s.width}))}});
+	if (s.bigram.buckets > 0) pl.push_back({&_bigram_table, {mat(tensor(0, TensorRole::Bigram, -1, {s.bigram.buckets + 1, s.width}))}});
 	if (s.depth_average) _scratch->hist_slabs = (int)s.layers.size() + 1;
 	if (s.embed_norm) pl.push_back({(void **)&_embed_norm, {vec32(s.norm_scalar ? tensor(0, TensorRole::EmbedNorm, -1, {}) : tensor(0, TensorRole::EmbedNorm, -1, {s.width}))}});
 	pl.push_back({&wcls, {mat(tensor(0, TensorRole::Head, -1, {s.vocab, s.width}))}});
@@ -366,6 +384,108 @@ void Model::build_stack(YALMData &data) {
 		auto L = std::make_shared<StackLayer>();
 		L->spec = s.layers[i];
 		const yalm::MixerSpec &m = L->spec.mix;
+		if (s.packed_block) {
+			// ---- one norm; one product in, [mixer's projections | gate | up | rest]; one product out, [W_o | W_down] ----
+			const int W = s.width;
+			const yalm::LayerSpec &ls = L->spec;
+			const FfnSpec &f = ls.ffn;
+			const int no = ls.mixed_width(), glu = f.kind == FfnSpec::Dense ? 2 * f.ff : 0;
+			pl.push_back({(void **)&L->norm1, {vec32(tensor(i, TensorRole::Norm1, -1, {W}))}});
+			pl.push_back({(void **)&L->norm1_bias, {vec32(tensor(i, TensorRole::Norm1Bias, -1, {W}))}});
+			Placement proj{&L->wproj, {}};
+			int at = 0; // columns of the product in so far
+			auto part = [&](TensorRole role, int rows) {
+				proj.parts.push_back(mat(tensor(i, role, -1, {rows, W})));
+				at += rows;
+				return at - rows;
+			};
+			auto feed_forward = [&] {
+				if (f.kind == FfnSpec::Dense) L->o_glu = part(TensorRole::Gate, f.ff), part(TensorRole::Up, f.ff);
+				else if (f.kind != FfnSpec::None) die("packed blocks take a dense feed-forward or none");
+			};
+			const Tensor *wo = nullptr;
+			if (ls.kind == yalm::MixerKind::DeltaRule) {
+				const yalm::DeltaSpec &d = ls.delta;
+				const int dk = d.kv_heads * d.dim, dv = d.heads * d.vdim, C = d.conv_channels();
+				if (!d.head_decay || !d.full_gate) die("packed blocks: the delta rule takes one decay per head and a full gate projection");
+				if (d.dim > 256) die("delta rule: key sizes above 256 are not built");
+				L->o_dq = part(TensorRole::DeltaQ, dk), part(TensorRole::DeltaK, dk), part(TensorRole::DeltaV, dv);
+				L->o_gate = part(TensorRole::DeltaGate, dv);
+				feed_forward();
+				L->o_beta = part(TensorRole::DeltaBeta, d.heads), L->o_a1 = part(TensorRole::DeltaDecay, d.heads);
+				pl.push_back({(void **)&L->conv_w, {vec32(tensor(i, TensorRole::DeltaQConv, -1, {dk, d.conv})), vec32(tensor(i, TensorRole::DeltaKConv, -1, {dk, d.conv})),
+				                                    vec32(tensor(i, TensorRole::DeltaVConv, -1, {dv, d.conv}))}});
+				pl.push_back({(void **)&L->d_a_log, {vec32(tensor(i, TensorRole::DeltaALog, -1, {d.heads}))}});
+				pl.push_back({(void **)&L->d_dt_bias, {vec32(tensor(i, TensorRole::DeltaDtBias, -1, {d.heads}))}});
+				pl.push_back({(void **)&L->d_norm, {vec32(tensor(i, TensorRole::DeltaNorm, -1, {d.vdim}))}});
+				wo = tensor(i, TensorRole::Wo, -1, {W, dv});
+				L->state_allocs.push_back({(void **)&L->conv_state, (size_t)d.conv * C * 4}); // a ring of the last `conv` positions' inputs
+				L->state_allocs.push_back({(void **)&L->scan_state, (size_t)d.heads * d.vdim * d.dim * 4});
+			} else if (ls.kind == yalm::MixerKind::TimeMix) {
+				const yalm::WkvSpec &k = ls.wkv;
+				const int hd = k.inner();
+				if (k.dim > 256) die("time mixing: head sizes above 256 are not built");
+				Placement mu{(void **)&L->mu, {}};
+				_host_converted.emplace_back((size_t)W * 4, 0);
+				const std::pair<const void *, size_t> zeros{_host_converted.back().data(), (size_t)W * 4};
+				auto segment = [&](TensorRole role) { // the columns so far end a segment that reads its own blend
+					mu.parts.push_back(vec32(tensor(i, role, -1, {W})));
+					L->seg_end.push_back(at);
+				};
+				L->o_q = part(TensorRole::WkvR, hd), segment(TensorRole::WkvMuR);
+				L->o_k = part(TensorRole::Wk, hd), segment(TensorRole::WkvMuK);
+				L->o_v = part(TensorRole::Wv, hd), segment(TensorRole::WkvMuV);
+				L->o_gate = part(TensorRole::OutGate, hd), segment(TensorRole::WkvMuG);
+				feed_forward();
+				if (glu) L->plain_mask = 1 << (int)L->seg_end.size(), mu.parts.push_back(zeros), L->seg_end.push_back(at);
+				L->o_a1 = part(TensorRole::WkvDecay1, k.decay_rank), segment(TensorRole::WkvMuW);
+				pl.push_back(mu);
+				pl.push_back({&L->wa2, {mat(tensor(i, TensorRole::WkvDecay2, -1, {hd, k.decay_rank}))}});
+				pl.push_back({(void **)&L->d_dt_bias, {vec32(tensor(i, TensorRole::WkvDecayBias, -1, {hd}))}});
+				pl.push_back({(void **)&L->bonus, {vec32(tensor(i, TensorRole::WkvBonus, -1, {k.heads, k.dim}))}});
+				pl.push_back({(void **)&L->mix_norm, {vec32(tensor(i, TensorRole::WkvNorm, -1, {hd}))}});
+				wo = tensor(i, TensorRole::Wo, -1, {W, hd});
+				L->state_allocs.push_back({(void **)&L->hprev, (size_t)2 * W * 4}); // the norm's output of the last two positions, slot = position & 1
+				L->state_allocs.push_back({(void **)&L->scan_state, (size_t)k.heads * k.dim * k.dim * 4});
+			} else if (ls.kind == yalm::MixerKind::Attention && m.qk_norm == yalm::QkNorm::PerHeadRotated && m.window == 0) {
+				const int nq = m.heads * m.dim, nk = m.kv_heads * m.dim, nv = m.kv_heads * m.vdim;
+				if (m.dim > 512 || m.vdim > 512) die("attention: head sizes above 512 are not built");
+				L->o_q = part(TensorRole::Wq, nq), L->o_k = part(TensorRole::Wk, nk), L->o_v = part(TensorRole::Wv, nv);
+				feed_forward();
+				pl.push_back({(void **)&L->qkb, {vec32(tensor(i, TensorRole::QBias, -1, {nq})), vec32(tensor(i, TensorRole::KBias, -1, {nk})), vec32(tensor(i, TensorRole::VBias, -1, {nv}))}});
+				if (m.sink) pl.push_back({(void **)&L->sink, {vec32(tensor(i, TensorRole::Sink, -1, {m.heads}))}});
+				wo = tensor(i, TensorRole::Wo, -1, {W, no});
+				if (m.rot.dims > 0) {
+					std::vector<float> fr;
+					m.rot.table(&fr, &L->rot_mag);
+					_host_converted.emplace_back(fr.size() * sizeof(float));
+					memcpy(_host_converted.back().data(), fr.data(), fr.size() * sizeof(float));
+					pl.push_back({(void **)&L->rot_freq, {{_host_converted.back().data(), fr.size() * sizeof(float)}}});
+				}
+				L->ring = c.max_seq_len;
+				const size_t cb = c.weight_dtype == DType::F32 ? 4 : 2;
+				L->state_allocs.push_back({&L->kring, (size_t)m.kv_heads * L->ring * m.dim * cb});
+				L->state_allocs.push_back({&L->vring, (size_t)m.kv_heads * L->ring * m.vdim * cb});
+			} else
+				die("packed blocks take the delta rule, time mixing, or causal attention with a norm after the rotation");
+			if (L->seg_end.empty() || L->seg_end.back() != at) L->seg_end.push_back(at);
+			if (ls.kind != yalm::MixerKind::TimeMix) L->plain_mask = 1;
+			pl.push_back(proj);
+			if (f.kind == FfnSpec::Dense) { // every output row's two weight rows side by side: one product over [mixer output | activation]
+				const auto a = mat(wo), b = mat(tensor(i, TensorRole::Down, -1, {W, f.ff}));
+				const size_t ra = a.second / W, rb = b.second / W;
+				_host_converted.emplace_back(a.second + b.second);
+				char *dst = _host_converted.back().data();
+				for (int r = 0; r < W; ++r) {
+					memcpy(dst + r * (ra + rb), static_cast<const char *>(a.first) + r * ra, ra);
+					memcpy(dst + r * (ra + rb) + ra, static_cast<const char *>(b.first) + r * rb, rb);
+				}
+				pl.push_back({&L->wout, {{dst, a.second + b.second}}});
+			} else
+				pl.push_back({&L->wout, {mat(wo)}});
+			_stack.push_back(L);
+			continue;
+		}
 		if (s.parallel_block) {
 			// ---- one norm, a packed projection of the mixer's input, per-mixer pieces, experts ----
 			const int W = s.width;
@@ -636,6 +756,25 @@ void Model::build_stack(YALMData &data) {
 		L->max_blocks = m.pool > 0 ? c.max_seq_len / m.pool + 1 : 0;
 		_stack.push_back(L);
 	}
+	if (s.loop_times > 1) { // repeated passes: the same weights (taken over after the upload), own caches and state
+		std::vector<std::shared_ptr<StackLayer>> runs;
+		std::vector<bool> used(_stack.size(), false);
+		for (const yalm::LayerRun &r : s.runs()) {
+			const StackLayer *first = _stack[r.layer].get();
+			if (first->kv_owner >= 0) die("repeated passes of a layer that shares its cache are not built");
+			auto L = _stack[r.layer];
+			if (used[r.layer]) {
+				L = std::make_shared<StackLayer>(*first);
+				L->shares = first;
+				for (auto &sa : L->state_allocs) // the same member of the copy
+					sa.first = reinterpret_cast<void **>(reinterpret_cast<char *>(L.get()) + (reinterpret_cast<const char *>(sa.first) - reinterpret_cast<const char *>(first)));
+			}
+			used[r.layer] = true;
+			L->add_embedding = r.add_embedding;
+			runs.push_back(L);
+		}
+		_stack = runs;
+	}
 	// v blending reads the first blending layer's values of the same rows: the shapes must agree
 	int first_nv = -1;
 	for (auto &L : _stack)
@@ -682,6 +821,14 @@ void Model::cuda_stack(int device) {
 			_device_bytes += part.second;
 		}
 	}
+	for (auto &L : _stack)
+		if (L->shares) { // weights are on the device now: take them over, keep what is this pass's own
+			const auto allocs = L->state_allocs;
+			const bool add = L->add_embedding;
+			const StackLayer *first = L->shares;
+			*L = *first;
+			L->state_allocs = allocs, L->add_embedding = add, L->shares = first;
+		}
 	for (auto &L : _stack) {
 		const yalm::MixerSpec &m = L->spec.mix;
 		for (auto &sa : L->state_allocs) {
@@ -733,6 +880,11 @@ void Model::cuda_stack(int device) {
 	const size_t kmax = std::max({W, (size_t)s.max_o_dim(), ff});
 	size_t shared_ff = 0;
 	for (const LayerSpec &l : s.layers) shared_ff = std::max<size_t>(shared_ff, l.ffn.shared_ff);
+	bool time_mix = false;
+	int mixes = 1;
+	for (auto &L : _stack)
+		if (L->spec.kind == yalm::MixerKind::TimeMix) time_mix = true, mixes = std::max(mixes, (int)L->seg_end.size());
+	const size_t blk = s.packed_block ? s.max_block_out() : 0;
 	const bool moe = s.max_experts() > 0 && c.weight_dtype != DType::F32; // the grouped route needs 16-bit operands
 	auto pad = [](size_t b) { return (b + 255) / 256 * 256; };
 	struct Slot {
@@ -742,12 +894,13 @@ void Model::cuda_stack(int device) {
 	             {(void **)&S.att, 4 * cap * std::max<size_t>(1, s.max_o_dim())},                   {(void **)&S.y, 4 * cap * top * W},
 	             {(void **)&S.gu, 4 * cap * 2 * ff},     {(void **)&S.h, 4 * cap * top * ff},    {(void **)&S.wts, 4 * cap * top},
 	             {(void **)&S.xn, 4 * cap * W},          {(void **)&S.logits, 4 * cap * (size_t)s.vocab}, {(void **)&S.probs, 4 * cap},
-	             {(void **)&S.a16, 2 * cap * top * kmax}, {(void **)&S.a16e, pb * 2 * cap * top * kmax}, {(void **)&S.a16r, pb * 2 * cap * top * kmax}, {(void **)&S.ids, 4 * cap * top},       {(void **)&S.tokens, 4 * cap},
+	             {(void **)&S.a16, 2 * cap * std::max({top * kmax, blk, mixes * W})}, {(void **)&S.a16e, pb * 2 * cap * top * kmax}, {(void **)&S.a16r, pb * 2 * cap * top * kmax}, {(void **)&S.ids, 4 * cap * top},       {(void **)&S.tokens, 4 * cap},
 	             {(void **)&S.want, 4 * cap},            {(void **)&S.targets, 4 * cap},
 	             {(void **)&S.attn_ws, 4 * yalm_attn_window_pool_workspace(512)}, {(void **)&S.ticket, 256},
 	             {(void **)&S.hs, pb * 4 * cap * W}, {(void **)&S.conv, pb * 4 * cap * nconv}, {(void **)&S.aux, pb * 4 * cap * naux},
 	             {(void **)&S.scan, pb * 4 * cap * no}, {(void **)&S.att2, pb * 4 * cap * no}, {(void **)&S.y1, pb * 4 * cap * W}, {(void **)&S.y2, pb * 4 * cap * W},
 	             {(void **)&S.hist, 4 * cap * W * (size_t)S.hist_slabs}, {(void **)&S.hsh, 4 * cap * shared_ff},
+	             {(void **)&S.mix, time_mix ? 4 * cap * mixes * W : 0}, {(void **)&S.blk, 4 * cap * blk}, {(void **)&S.x0, s.loop_times > 1 ? 4 * cap * W : 0}, {(void **)&S.prev, 256},
 	             {(void **)&S.lat16, lat16}, {(void **)&S.latkv, latkv}, {(void **)&S.lat_ek, lat_ek}, {(void **)&S.lat_ev, lat_ev},
 	             {(void **)&S.moe_gu, moe ? 4 * cap * top * 2 * ff : 0}, {(void **)&S.moe_ys, moe ? 4 * cap * top * W : 0}, {(void **)&S.order, 4 * cap * top}};
 	size_t total = 0;
@@ -771,11 +924,14 @@ void Model::cuda_stack(int device) {
 // y = alpha * x W^T.  16-bit weights and enough rows: activations rounded once to the weight type, product on the tcgen05
 // tensor cores (prefill_gemm.cu); otherwise (fp32 mode, few rows, rows that are not 16-byte multiples) the SIMT routes,
 // which keep the activations in fp32.
+static bool tc_off() { // YALM_STACK_TC=0: A/B against the SIMT products
+	static const bool off = [] { const char *e = getenv("YALM_STACK_TC"); return e && e[0] == '0'; }();
+	return off;
+}
 static int stack_linear(Model &, const Config &c, void *a16, float *y, int ldy, const float *x, int ldx, const void *w, int M, int N, int K,
                         float alpha, cudaStream_t st) {
 	const int dt = static_cast<int>(c.weight_dtype);
-	static const bool tc_off = [] { const char *e = getenv("YALM_STACK_TC"); return e && e[0] == '0'; }();
-	if (!tc_off && dt != YALM_F32 && M >= 32 && K % 8 == 0 && K >= 8 && ldy % 4 == 0 && ((uintptr_t)y & 15) == 0 && ((uintptr_t)w & 15) == 0) {
+	if (!tc_off() && dt != YALM_F32 && M >= 32 && K % 8 == 0 && K >= 8 && ldy % 4 == 0 && ((uintptr_t)y & 15) == 0 && ((uintptr_t)w & 15) == 0) {
 		ST_TRY(yalm_cast_rows16(a16, x, ldx, M, K, dt == YALM_BF16, st));
 		return yalm_gemm_16(y, ldy, a16, w, M, N, K, 0, dt == YALM_BF16, alpha, st);
 	}
@@ -1095,6 +1251,99 @@ int Model::stack_layer_prenorm(StackScratch &S, const yalm::StackLayer &L, int i
 	return yalm_residual_sum_rows(S.x, add_a, add_b, slots, W, nsum, n, W, st);
 }
 
+// One parallel block over n rows, x += mixer(h) + ff(h) with h = N(x): ONE product of h gives the mixer's projections and the
+// feed-forward's gate and up, ONE product over [mixer output | activation] is added to x.  A decode row is three launches for a matrix-state
+// mixer (five for attention): the norm — and time mixing's blends, by output segment — while the first product stages its input,
+// the mixer, and the activation while the second stages its input with x += in its epilogue.  What the rows leave for the next
+// call (convolution inputs, the previous h, matrix states, keys and values) is written by the ops themselves.
+int Model::stack_layer_block(StackScratch &S, const yalm::StackLayer &L, const yalm::StackLayer *next, int n, int pos0, const int *ctl, cudaStream_t st) {
+	const Config &c = *config;
+	const StackSpec &sp = *c.stack;
+	const yalm::LayerSpec &ls = L.spec;
+	const FfnSpec &f = ls.ffn;
+	const int dt = static_cast<int>(c.weight_dtype), W = sp.width, f32 = c.weight_dtype == DType::F32, bf16 = c.weight_dtype == DType::BF16;
+	const int ldp = ls.proj_width(), ncols = L.seg_end.back(), no = ls.mixed_width(), ff = f.kind == FfnSpec::Dense ? f.ff : 0, K2 = no + ff, act = glu_act_code(f.act);
+	const int nseg = (int)L.seg_end.size();
+	const bool mixes = ls.kind == yalm::MixerKind::TimeMix;
+	float *P = S.qkv;
+	const bool fuse = gemv_fusable(c, n, W, L.wproj, S.x) && gemv_fusable(c, n, K2, L.wout, S.x) && no % 4 == 0 && ff % 4 == 0 && L.o_glu % 4 == 0;
+	bool bounds4 = true;
+	for (int e = 0; e + 1 < nseg; ++e) bounds4 = bounds4 && L.seg_end[e] % 4 == 0;
+	const bool tc = !fuse && !f32 && !tc_off() && n >= 32 && W % 8 == 0 && K2 % 8 == 0 && bounds4 && ((uintptr_t)L.wproj & 15) == 0 && ((uintptr_t)L.wout & 15) == 0;
+	const float *add = L.add_embedding && !S.x0_added ? S.x0 : nullptr;
+	S.x0_added = false;
+	// ---- product in ----
+	if (fuse) {
+		if (add) ST_TRY(yalm_residual_sum_rows(S.x, add, nullptr, nullptr, 0, 0, n, W, st));
+		ST_TRY(yalm_gemv_block_in(P, S.x, L.wproj, W, ncols, dt, L.norm1, L.norm1_bias, sp.norm_eps, nseg, L.seg_end.data(), L.mu, L.plain_mask, L.hprev, pos0, ctl, st));
+	} else {
+		const bool direct = tc && !mixes; // the norm's output is the tensor-core operand itself
+		ST_TRY(yalm_layer_norm_rows(direct ? nullptr : S.xn, direct ? S.a16 : nullptr, bf16, S.x, add, nullptr, L.norm1, L.norm1_bias, sp.norm_eps, n, W, st));
+		if (mixes) ST_TRY(yalm_mix_rows(tc ? nullptr : S.mix, tc ? S.a16 : nullptr, bf16, S.xn, L.mu, nseg, L.plain_mask, L.hprev, n, W, pos0, ctl, st));
+		if (tc)
+			ST_TRY(yalm_gemm_16_segments(P, ldp, S.a16, L.wproj, n, ncols, W, nseg, L.seg_end.data(), bf16, st));
+		else
+			for (int e = 0, at = 0; e < nseg; at = L.seg_end[e++])
+				ST_TRY(stack_linear(*this, c, S.a16, P + at, ldp, mixes ? S.mix + (size_t)e * n * W : S.xn, W,
+				                    static_cast<const char *>(L.wproj) + (size_t)at * W * dtype_size(c.weight_dtype), n, L.seg_end[e] - at, W, 1.f, st));
+	}
+	// ---- mixer ----
+	const float *o = S.scan, *norm_w = nullptr; // what the output product's input is made from: heads x vdim columns, normed and gated when norm_w is set
+	int w_stride = 0, heads = 0;
+	if (ls.kind == yalm::MixerKind::DeltaRule) {
+		const yalm::DeltaSpec &d = ls.delta;
+		const int dk = d.kv_heads * d.dim, dv = d.heads * d.vdim, C = d.conv_channels(), H = d.heads;
+		const float q_scale = 1.0f / sqrtf((float)d.dim);
+		heads = H, norm_w = L.d_norm;
+		if (fuse)
+			ST_TRY(yalm_delta_step(S.att, L.scan_state, P, L.o_dq, L.o_gate, L.o_beta, L.o_a1, L.conv_w, L.conv_state, L.d_a_log, L.d_dt_bias, L.d_norm, H, d.kv_heads, d.dim,
+			                       d.vdim, d.conv, 1e-6f, q_scale, sp.norm_eps, pos0, ctl, st));
+		else {
+			ST_TRY(yalm_delta_in_rows(S.conv, S.aux, P + L.o_dq, P + L.o_beta, ldp, L.conv_w, L.conv_state, L.d_a_log, L.d_dt_bias, n, H, d.kv_heads, d.dim, d.vdim, d.conv,
+			                          1e-6f, q_scale, pos0, ctl, st));
+			ST_TRY(yalm_state_scan_rows(S.scan, dv, S.conv + dk, C, S.conv, C, S.conv + 2 * dk, C, S.aux, 2 * H, 0, nullptr, 0, S.aux + H, 2 * H, nullptr, L.scan_state, n, H,
+			                            H / d.kv_heads, d.dim, d.vdim, pos0, ctl, st));
+		}
+	} else if (mixes) {
+		const yalm::WkvSpec &k = ls.wkv;
+		const int hd = k.inner();
+		heads = k.heads, norm_w = L.mix_norm, w_stride = k.dim;
+		if (fuse)
+			ST_TRY(yalm_wkv_step(S.att, L.scan_state, P, L.o_q, L.o_k, L.o_v, L.o_gate, L.o_a1, L.wa2, L.d_dt_bias, L.bonus, L.mix_norm, dt, k.heads, k.dim, k.decay_rank,
+			                     sp.norm_eps, pos0, ctl, st));
+		else {
+			ST_TRY(yalm_wkv_decay_rows(S.aux, hd, P + L.o_a1, ldp, L.wa2, L.d_dt_bias, dt, n, hd, k.decay_rank, st));
+			ST_TRY(yalm_state_scan_bonus_rows(S.scan, hd, P + L.o_k, ldp, P + L.o_q, ldp, P + L.o_v, ldp, S.aux, hd, L.bonus, L.scan_state, n, k.heads, k.dim, k.dim, pos0,
+			                                  ctl, st));
+		}
+	} else {
+		const yalm::MixerSpec &m = ls.mix;
+		const int nq = m.heads * m.dim, nk = m.kv_heads * m.dim;
+		heads = m.heads, o = S.att;
+		ST_TRY(yalm_head_bias_rope_norm_append_rows(P, ldp, L.o_q, L.o_k, L.o_v, m.heads, m.kv_heads, m.kv_heads, m.dim, m.vdim, L.qkb, L.qkb + nq, L.qkb + nq + nk, L.rot_freq,
+		                                            L.rot_mag, m.rot.dims, m.rot.interleaved ? 1 : 0, sp.norm_eps, L.kring, L.vring, L.ring, f32, n, pos0, ctl, st));
+		// many rows over bf16 rings: tensor-core attention; decode-sized calls, the fp32 cache and other head sizes: the SIMT kernels
+		if (!f32 && n >= 16 && no % 2 == 0 && yalm_attn_window_pool_mma_shape(m.dim, m.vdim) && !attn_mma_off())
+			ST_TRY(yalm_attn_window_pool_mma_sink(S.att, no, P + L.o_q, ldp, L.kring, L.vring, nullptr, nullptr, n, m.heads, m.kv_heads, m.dim, m.vdim, L.ring, 0, 0, 0, m.scale,
+			                                      pos0, ctl, L.sink, m.kv_heads, st));
+		else
+			ST_TRY(yalm_attn_window_pool_sink(S.att, no, P + L.o_q, ldp, L.kring, m.dim, L.vring, m.vdim, nullptr, nullptr, S.attn_ws, n, m.heads, m.kv_heads, m.dim, m.vdim, L.ring,
+			                                  0, 0, 0, m.scale, f32, c.max_seq_len, pos0, ctl, L.sink, m.kv_heads, st));
+	}
+	// ---- product out, x += ----
+	if (fuse) {
+		const bool pass_starts = next && next->add_embedding && !_stack_tap; // a tap reads x between the two additions
+		ST_TRY(yalm_gemv_block_out(S.x, S.att, no, P + L.o_glu, ff, act, L.wout, W, dt, pass_starts ? S.x0 : nullptr, st));
+		S.x0_added = pass_starts;
+		return 0;
+	}
+	ST_TRY(yalm_block_out_rows(tc ? nullptr : S.blk, tc ? S.a16 : nullptr, bf16, K2, o, no, norm_w ? P + L.o_gate : nullptr, P + L.o_glu, ldp, norm_w, w_stride, sp.norm_eps, n,
+	                           heads, no / heads, ff, act, st));
+	if (tc) return yalm_gemm_16(S.x, W, S.a16, L.wout, n, W, K2, 1, bf16, 1.f, st);
+	ST_TRY(stack_linear(*this, c, S.a16, S.y1, W, S.blk, K2, L.wout, n, W, K2, 1.f, st));
+	return yalm_residual_sum_rows(S.x, S.y1, nullptr, nullptr, 0, 0, n, W, st);
+}
+
 static int plain_act_code(yalm::GluAct a) {
 	return a == yalm::GluAct::GeluErf ? 4 : a == yalm::GluAct::GeluTanh ? 3 : a == yalm::GluAct::Silu ? YALM_ACT_SILU : YALM_ACT_GELU;
 }
@@ -1252,7 +1501,13 @@ int Model::stack_pass(InferenceState &s, int n, int pos0, bool from_ctl, int n_w
 	const int dt = static_cast<int>(c.weight_dtype), W = sp.width, f32 = c.weight_dtype == DType::F32;
 	const int *ctl = from_ctl ? s.ctl() : nullptr;
 	const float woff = sp.norm_one_plus ? 1.f : 0.f;
-	ST_TRY(yalm_embed_rows(S.x, token_embedding_table, _pos_table, dt, from_ctl ? nullptr : S.tokens, n, W, pos0, ctl, sp.embed_scale, st));
+	if (sp.bigram.buckets > 0)
+		ST_TRY(yalm_embed_bigram_rows(S.x, S.x0, token_embedding_table, _bigram_table, dt, from_ctl ? nullptr : S.tokens, sp.bigram.buckets, sp.bigram.mul_prev,
+		                              sp.bigram.mul_cur, S.prev, n, W, pos0, ctl, st));
+	else {
+		ST_TRY(yalm_embed_rows(S.x, token_embedding_table, _pos_table, dt, from_ctl ? nullptr : S.tokens, n, W, pos0, ctl, sp.embed_scale, st));
+		if (S.x0) ST_TRY(cudaMemcpyAsync(S.x0, S.x, sizeof(float) * n * W, cudaMemcpyDeviceToDevice, st));
+	}
 	if (sp.embed_norm) ST_TRY(yalm_norm_shift_rows(S.x, nullptr, S.x, _embed_norm, sp.norm_scalar, woff, sp.norm_eps, nullptr, nullptr, n, W, pos0, ctl, st));
 	if (sp.depth_average) ST_TRY(yalm_depth_average_rows(S.x, S.hist, (size_t)S.cap * W, nullptr, 1, n, W, nullptr, nullptr, nullptr, 0, 0, st)); // slab 0: the embedding output
 	int layer_no = 0;
@@ -1264,10 +1519,15 @@ int Model::stack_pass(InferenceState &s, int n, int pos0, bool from_ctl, int n_w
 		++layer_no;
 		return 0;
 	};
-	S.xn_valid = false;
+	S.xn_valid = S.x0_added = false;
 	for (size_t li = 0; li < _stack.size(); ++li) {
 		auto &Lp = _stack[li];
 		const StackLayer &L = *Lp;
+		if (sp.packed_block) {
+			ST_TRY(stack_layer_block(S, L, li + 1 < _stack.size() ? _stack[li + 1].get() : nullptr, n, pos0, ctl, st));
+			ST_TRY(tap());
+			continue;
+		}
 		if (sp.parallel_block) {
 			ST_TRY(stack_layer_parallel(S, L, n, pos0, ctl, st));
 			ST_TRY(tap());
@@ -1337,7 +1597,11 @@ int Model::stack_pass(InferenceState &s, int n, int pos0, bool from_ctl, int n_w
 		ST_TRY(tap());
 	}
 	if (n_want > 0) {
-		if (sp.layer_norm)
+		if (sp.norm_bias && n_want == 1 && sp.logit_scale == 1.f && !(sp.logit_softcap > 0.f) && gemv_fusable(c, n, W, wcls, S.x)) // a decode row: norm + head as one launch
+			return yalm_gemv_block_in(s.logits_dev(), S.x, wcls, W, sp.vocab, dt, rms_final_weight, _final_bias, sp.norm_eps, 1, nullptr, nullptr, 1, nullptr, pos0, ctl, st);
+		if (sp.norm_bias)
+			ST_TRY(yalm_layer_norm_rows(S.xn, nullptr, 0, S.x, nullptr, from_ctl ? nullptr : S.want, rms_final_weight, _final_bias, sp.norm_eps, n_want, W, st));
+		else if (sp.layer_norm)
 			ST_TRY(yalm_layer_norm_gather_rows(S.xn, S.x, from_ctl ? nullptr : S.want, rms_final_weight, 1, sp.norm_eps, n_want, W, st));
 		else
 			ST_TRY(yalm_norm_gather_rows(S.xn, S.x, from_ctl ? nullptr : S.want, rms_final_weight, sp.norm_scalar, woff, sp.norm_eps, n_want, W, st));

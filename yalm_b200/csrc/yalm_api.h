@@ -293,7 +293,7 @@ struct Model {
 	int stack_read(int layer, int which, float *dst, size_t count);
 	int stack_ring_slots(int layer) const;
 	// Tests: after every layer of the next passes, the residual rows (n, width) are copied to dst + layer * n * width
-	// (host, n_layers * n * width floats for calls of n <= stack_chunk rows); null switches it off.
+	// (host, layer runs * n * width floats — a layer that runs several times counts each time — for calls of n <= stack_chunk rows); null switches it off.
 	void stack_tap(float *dst) { _stack_tap = dst; }
 	size_t device_bytes() const { return _device_bytes; }
 	// loader facts for tests / bench: number of device allocations behind the model (1) and whether the upload went through pinned staging
@@ -326,6 +326,8 @@ private:
 	float *_embed_norm = nullptr;                   // weight of the norm after the embedding, when the design has one
 	void *_pos_table = nullptr;                     // learned positions (max_positions, dim), weight dtype
 	void *_side_table = nullptr;                    // second token embedding (vocab, layers * token_side), weight dtype
+	void *_bigram_table = nullptr;                  // bigram embedding (buckets + 1, dim), weight dtype
+	float *_final_bias = nullptr;                   // bias of the final norm, when the design has one
 	std::vector<std::vector<char>> _host_converted; // weights converted on the host (bf16 -> fp32, norm weights), alive until the upload
 	struct StackScratch;
 	std::shared_ptr<StackScratch> _scratch;
@@ -339,6 +341,7 @@ private:
 	int stack_pass(InferenceState &s, int n, int pos0, bool from_ctl, int n_want);
 	int stack_moe_grouped(StackScratch &S, const yalm::StackLayer &L, const float *x, void *a16, int n, int act, cudaStream_t st);
 	int stack_layer_parallel(StackScratch &S, const yalm::StackLayer &L, int n, int pos0, const int *ctl, cudaStream_t st);
+	int stack_layer_block(StackScratch &S, const yalm::StackLayer &L, const yalm::StackLayer *next, int n, int pos0, const int *ctl, cudaStream_t st);
 	int stack_layer_prenorm(StackScratch &S, const yalm::StackLayer &L, int index, int n, int pos0, const int *ctl, cudaStream_t st);
 	int stack_layer_sandwich(StackScratch &S, const yalm::StackLayer &L, const yalm::StackLayer *next, int index, int n, int pos0, const int *ctl, bool from_ctl,
 	                         cudaStream_t st);
