@@ -580,6 +580,178 @@ def run_kiduvik(args, base, emit, shm_path, ClockSampler):
                           l2="inputs larger than L2 (weights streamed per token)")))
 
 
+# ---- Fafelix ---------------------------------------------------------------------------------------------------------------
+# name: width; causal attention heads / kv heads / head size; delta rule heads / kv heads x (dim, vdim); time mixing heads x dim and the
+# decay's rank; feed-forward; layer order (d = delta rule, a = attention, t = time mixing) and the span that runs several times
+FAFELIX_SIZES = {
+    "w2048": dict(width=2048, heads=16, kv_heads=4, dim=128, dheads=16, dkv=8, ddim=128, dvdim=128, theads=32, tdim=64, rank=64, ff=8192, order="dtad", loop=None,
+                  vocab=32000),
+    "w4096": dict(width=4096, heads=32, kv_heads=8, dim=128, dheads=32, dkv=16, ddim=128, dvdim=128, theads=64, tdim=64, rank=64, ff=14336, order="dat", loop=(1, 3, 2),
+                  vocab=32000),
+}
+
+
+def fafelix_runs(z):
+    """Layer kinds in the order they run."""
+    o = z["order"]
+    if not z["loop"]:
+        return o
+    a, b, times = z["loop"]
+    return o[:a] + o[a:b] * times + o[b:]
+
+
+def write_fafelix(folder, z):
+    """A checkpoint directory of the given size: matrices tiled from one random block, norm weights 1."""
+    os.makedirs(folder, exist_ok=True)
+    rng = np.random.default_rng(6)
+    block = _bf16(rng.standard_normal(1 << 22).astype(np.float32) * 0.02)
+    W, conv = z["width"], 4
+    mlp = {"kind": "dense", "ff": z["ff"]}
+    kinds = {"d": {"type": "delta", "mlp": mlp, "mixer": {"heads": z["dheads"], "kv_heads": z["dkv"], "dim": z["ddim"], "vdim": z["dvdim"], "conv": conv}},
+             "a": {"type": "attention", "mlp": mlp, "mixer": {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["dim"], "scale": z["dim"] ** -0.5,
+                                                             "rot": {"base": 10000.0, "dims": z["dim"] // 2,
+                                                                     "scaling": {"factor": 4.0, "low": 1.0, "high": 2.0, "original": 2048}}}},
+             "t": {"type": "wkv", "mlp": mlp, "mixer": {"heads": z["theads"], "dim": z["tdim"]}}}
+    cfg = {"architecture": "Fafelix", "width": W, "vocab": z["vocab"], "norm": {"eps": 1e-5},
+           "embedding": {"bigram": {"buckets": 8191, "mul_prev": 1009, "mul_cur": 31}}, "layers": [kinds[c] for c in z["order"]]}
+    if z["loop"]:
+        cfg["loop"] = dict(zip(("start", "stop", "times"), z["loop"]))
+    with open(os.path.join(folder, "config.json"), "w") as f:
+        json.dump(cfg, f)
+    shapes = {"embed": (z["vocab"], W), "bigram": (8192, W), "final.norm": (W,), "final.norm.b": (W,), "head": (z["vocab"], W)}
+    for i, c in enumerate(z["order"]):
+        p, m, f = "l%d." % i, "l%d.mix." % i, "l%d.mlp." % i
+        shapes.update({p + "norm1": (W,), p + "norm1.b": (W,), f + "gate": (z["ff"], W), f + "up": (z["ff"], W), f + "down": (W, z["ff"])})
+        if c == "d":
+            H, dk, dv = z["dheads"], z["dkv"] * z["ddim"], z["dheads"] * z["dvdim"]
+            for n, ch in (("q", dk), ("k", dk), ("v", dv)):
+                shapes.update({m + n: (ch, W), m + n + ".conv": (ch, conv)})
+            shapes.update({m + "b": (H, W), m + "a": (H, W), m + "A_log": (H,), m + "dt_bias": (H,), m + "norm": (z["dvdim"],), m + "g": (dv, W), m + "o": (W, dv)})
+        elif c == "a":
+            nq, nk = z["heads"] * z["dim"], z["kv_heads"] * z["dim"]
+            shapes.update({m + "q": (nq, W), m + "q.b": (nq,), m + "k": (nk, W), m + "k.b": (nk,), m + "v": (nk, W), m + "v.b": (nk,), m + "sink": (z["heads"],), m + "o": (W, nq)})
+        else:
+            hd = z["theads"] * z["tdim"]
+            shapes.update({m + "mu." + s: (W,) for s in "rkvgw"})
+            shapes.update({m + s: (hd, W) for s in "rkvg"})
+            shapes.update({m + "w1": (z["rank"], W), m + "w2": (hd, z["rank"]), m + "w0": (hd,), m + "u": (z["theads"], z["tdim"]), m + "norm": (hd,), m + "o": (W, hd)})
+    header, off = {}, 0
+    for name, shp in shapes.items():
+        n = int(np.prod(shp))
+        header[name] = {"dtype": "BF16", "shape": list(shp), "data_offsets": [off, off + 2 * n]}
+        off += 2 * n
+    h = json.dumps(header).encode()
+    h += b" " * (-len(h) % 8)
+    one = _bf16(np.ones(1, np.float32))[0]
+    with open(os.path.join(folder, "model.safetensors"), "wb") as f:
+        f.write(struct.pack("<Q", len(h)) + h)
+        for k, (name, shp) in enumerate(shapes.items()):
+            n = int(np.prod(shp))
+            if name.endswith("norm") or name.endswith("norm1"):
+                f.write(np.full(n, one, np.uint16).tobytes())
+            elif len(shp) < 2:
+                f.write(block[:n].tobytes())
+            else:
+                f.write(np.resize(np.roll(block, 7919 * k), n).tobytes())
+    return cfg
+
+
+def fafelix_numbers(z):
+    """-> (decode bytes per token at CONTEXT, prefill FLOP per token), every layer run counted: its matrices once (bf16), the fp32 matrix
+    states read and written, all earlier keys and values; 2 FLOP per parameter plus the attention's products over the causal half
+    of the context and the recurrences' own (decay, two products, update: 8 per state element of the delta rule, 6 of the time mixing)."""
+    W = z["width"]
+    params, state, extra = z["vocab"] * W, 0, 0.0
+    for c in fafelix_runs(z):
+        params += 3 * z["ff"] * W
+        if c == "d":
+            dk, dv = z["dkv"] * z["ddim"], z["dheads"] * z["dvdim"]
+            params += (2 * dk + 3 * dv + 2 * z["dheads"]) * W
+            state += 2 * 4 * z["dheads"] * z["ddim"] * z["dvdim"]
+            extra += 8.0 * z["dheads"] * z["ddim"] * z["dvdim"]
+        elif c == "a":
+            nq, nk = z["heads"] * z["dim"], z["kv_heads"] * z["dim"]
+            params += (2 * nq + 2 * nk) * W
+            state += CONTEXT * 2 * nk * 2
+            extra += 4.0 * nq * CONTEXT / 2
+        else:
+            hd = z["theads"] * z["tdim"]
+            params += (5 * hd + z["rank"]) * W + hd * z["rank"]
+            state += 2 * 4 * hd * z["tdim"]
+            extra += 6.0 * hd * z["tdim"]
+    return 2 * params + state, 2.0 * (params - z["vocab"] * W) + extra
+
+
+def run_fafelix(args, base, emit, shm_path, ClockSampler):
+    """`bench.py --workload fafelix-sizes`: the Fafelix design beside the closest existing models on the same executor: the dense Retezen
+    stack (attention over the whole context, dense feed-forward) at equal width, heads, feed-forward, layer runs and vocabulary, and, for
+    the recurrence, Fapudra (parallel blocks with a delta rule)."""
+    import torch
+    from yalm_b200 import api
+    pk = os.path.join(ROOT, "MEASURED_PEAKS.json")
+    peaks = json.load(open(pk)) if os.path.exists(pk) else {"hbm_gbs": 6650.0, "bf16_tflops_sustained": 1400.0}
+    hbm, tflops = float(peaks["hbm_gbs"]), float(peaks["bf16_tflops_sustained"])
+    steps = max(8, min(args.steps, 128))
+    clocks = ClockSampler(0)
+    clocks.start()
+    out, launches = [], 0
+
+    def measure(model, ids):
+        st = api.InferenceState(model)
+        st.forward_batch(ids[:1024], 0)                     # warm-up (sizes kernels, first-use set-up)
+        st.end_sequence()
+        torch.cuda.synchronize()
+        t0 = time.perf_counter()
+        st.forward_batch(ids[:-1], 0)
+        t_pre = time.perf_counter() - t0
+        st.generate_greedy(ids[-1], CONTEXT - 1, max(3, args.warmup))   # first step eager + graph capture, untimed
+        st.generate_greedy(ids[0], CONTEXT - 1 + max(3, args.warmup), steps)
+        t_dec = st.device_ms / 1e3
+        n = model.launches()
+        st.close()
+        return (CONTEXT - 1) / t_pre, steps / t_dec, n
+
+    def line(write, context, numbers, ids):
+        folder = shm_path("yalm_bench_fafelix_%d" % os.getpid())
+        try:
+            write(folder)
+            model = api.Model(folder, context, api.BF16).cuda(0)
+        finally:
+            shutil.rmtree(folder, ignore_errors=True)
+        pre, dec, n = measure(model, ids)
+        model.close()
+        dec_bytes, pre_flop = numbers
+        return {"prefill_tok_s": pre, "decode_tok_s": dec, "prefill_frac_of_measured_bf16": pre_flop * pre / 1e12 / tflops,
+                "decode_frac_of_measured_hbm": dec_bytes * dec / 1e9 / hbm, "decode_bytes_per_token": dec_bytes, "launches_per_token": n}
+
+    only = os.environ.get("YALM_BENCH_SIZES", "").split(",") if os.environ.get("YALM_BENCH_SIZES") else None
+    ctx = CONTEXT + steps + args.warmup + 8
+    for name, z in FAFELIX_SIZES.items():
+        if only and name not in only:
+            continue
+        ids = [(i * 7919 + 1) % z["vocab"] for i in range(CONTEXT)]
+        row = {"size": name, "width": z["width"], "layer_runs": fafelix_runs(z), "context": CONTEXT}
+        row["fafelix"] = line(lambda f: write_fafelix(f, z), ctx, fafelix_numbers(z), ids)
+        launches += steps * row["fafelix"]["launches_per_token"]
+        if not os.environ.get("YALM_BENCH_NO_PEER"):
+            zr = dict(SIZES[name], layers=len(fafelix_runs(z)), window=0, pool=0)       # window 0: the whole context, as here
+            _, r_bytes, r_flop = retezen_numbers(dict(zr, window=CONTEXT, pool=64), "dense")
+            r_flop -= 4.0 * zr["layers"] * zr["heads"] * zr["dim"] * CONTEXT / 2       # the causal half
+            row["equal_size_retezen"] = line(lambda f: write_retezen(f, zr, "dense", ctx), 0, (r_bytes, r_flop), ids)
+            if name in FAPUDRA_SIZES:
+                zf = FAPUDRA_SIZES[name]
+                row["equal_width_fapudra"] = line(lambda f: write_fapudra(f, zf, ctx), 0, fapudra_numbers(zf), ids)
+        out.append(row)
+    clk = clocks.stop()
+    first = out[0]["fafelix"]
+    emit(dict(base, impl="ours", metric="batch-1 decode tok/s (Fafelix, first size; all sizes under `sizes`)", value=first["decode_tok_s"], steps=steps,
+              ms_per_step=1000.0 / first["decode_tok_s"], dtype="bf16", clocks=clk, gpu_launches=launches, sizes=out,
+              e2e={"value": first["decode_tok_s"], "unit": "tok/s", "h2d_bytes_per_step": 0, "d2h_bytes_per_step": 4,
+                   "note": "device loop: token ids stay on the device, 4 bytes per token come back"},
+              config=dict(base["config"], workload="Fafelix at model-like sizes beside the equal-size dense Retezen stack", context=CONTEXT,
+                          l2="inputs larger than L2 (weights streamed per token)")))
+
+
 def run(args, base, emit, write_yalm, shm_path, ClockSampler):
     import torch
     from yalm_b200 import api
