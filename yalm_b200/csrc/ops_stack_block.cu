@@ -294,7 +294,7 @@ __global__ void __launch_bounds__(256) block_out_rows_kernel(BlockOutArgs a) {
 // ---- a decode row of a matrix-state mixer ---------------------------------------------------------------------------------------
 // One CTA per head: (DELTA) convolution + SiLU + unit norms of the head's q and k and of its P channels of v, decay and beta; or
 // (time mixing) the decay's second stage for the head's D channels.  Then one step of the recurrence with the state in the layout
-// and the order of sums of state_scan_kernel (8 lanes per column, EPL consecutive rows each), the head's RMS norm, weight and gate.
+// of state_scan_kernel (8 lanes per column, EPL consecutive rows each), the head's RMS norm, weight and gate.
 struct StateStepArgs {
 	float *out;                   // (H P)
 	float *state;                 // (H, P, D)
@@ -503,7 +503,11 @@ __global__ void __launch_bounds__(kBlockThreads) gemv_block_kernel(GemvBlockArgs
 			}
 	};
 	if constexpr (!IN) {
+		const int ntasks = (a.d + R - 1) / R;
+		const int first = blockIdx.x * nw + warp;
+#pragma unroll 4
 		for (int e = threadIdx.x * 4; e < a.n1; e += blockDim.x * 4) *reinterpret_cast<float4 *>(xs + xs_slot<EP>(e)) = *reinterpret_cast<const float4 *>(a.x1 + e);
+#pragma unroll 4
 		for (int e = threadIdx.x * 4; e < a.ff; e += blockDim.x * 4) {
 			const float4 g = *reinterpret_cast<const float4 *>(a.gu + e), u = *reinterpret_cast<const float4 *>(a.gu + a.ff + e);
 			*reinterpret_cast<float4 *>(xs + xs_slot<EP>(a.n1 + e)) =
@@ -511,9 +515,12 @@ __global__ void __launch_bounds__(kBlockThreads) gemv_block_kernel(GemvBlockArgs
 			                glu_value(g.w, u.w, a.act, 1.f, 0.f, 0.f));
 		}
 		__syncthreads();
-		const int ntasks = (a.d + R - 1) / R;
-		for (int t = blockIdx.x * nw + warp; t < ntasks; t += gridDim.x * nw) rows(t * R, a.d);
+		for (int t = first; t < ntasks; t += gridDim.x * nw) rows(t * R, a.d);
 	} else {
+		// row groups never straddle two segments; this CTA's range [t0, t1) of all groups
+		int total = 0;
+		for (int g = 0, at = 0; g < a.nseg; ++g) total += (a.seg_end[g] - at + R - 1) / R, at = a.seg_end[g];
+		const int t0 = (int)((long long)blockIdx.x * total / gridDim.x), t1 = (int)((long long)(blockIdx.x + 1) * total / gridDim.x);
 		float s = 0.f;
 #pragma unroll 4
 		for (int e = threadIdx.x * 4; e < a.n; e += blockDim.x * 4) {
@@ -534,6 +541,7 @@ __global__ void __launch_bounds__(kBlockThreads) gemv_block_kernel(GemvBlockArgs
 		auto stage = [&](int seg) {
 			const bool mix = !((a.plain >> seg) & 1);
 			float *keep = a.state && blockIdx.x == 0 ? a.state + (size_t)(p & 1) * a.n : nullptr;
+#pragma unroll 2
 			for (int e = threadIdx.x * 4; e < a.n; e += blockDim.x * 4) {
 				const float4 v = *reinterpret_cast<const float4 *>(a.x + e), g = *reinterpret_cast<const float4 *>(a.nw + e), b = *reinterpret_cast<const float4 *>(a.nb + e);
 				float4 o = make_float4((v.x - mean) * sc * g.x + b.x, (v.y - mean) * sc * g.y + b.y, (v.z - mean) * sc * g.z + b.z, (v.w - mean) * sc * g.w + b.w);
@@ -546,10 +554,6 @@ __global__ void __launch_bounds__(kBlockThreads) gemv_block_kernel(GemvBlockArgs
 				*reinterpret_cast<float4 *>(xs + xs_slot<EP>(e)) = o;
 			}
 		};
-		// row groups never straddle two segments; this CTA's range [t0, t1) of all groups
-		int total = 0;
-		for (int g = 0, at = 0; g < a.nseg; ++g) total += (a.seg_end[g] - at + R - 1) / R, at = a.seg_end[g];
-		const int t0 = (int)((long long)blockIdx.x * total / gridDim.x), t1 = (int)((long long)(blockIdx.x + 1) * total / gridDim.x);
 		int base = 0, start = 0; // first group and first row of the segment
 		for (int g = 0; g < a.nseg; ++g) {
 			const int groups = (a.seg_end[g] - start + R - 1) / R;
@@ -570,8 +574,9 @@ static int launch_gemv_block(const GemvBlockArgs &a, int dtype, cudaStream_t st)
 	const int ep = dtype == YALM_F32 ? 4 : 8, ch = 32 * ep;
 	const size_t smem = (36 + (size_t)((a.n + ch - 1) / ch * ch)) * sizeof(float);
 	if (!a.w || a.n < 1 || a.d < 1 || a.n % ep || ((uintptr_t)a.w & 15) || (int)smem > device_info().max_smem_optin) return YALM_EINVAL;
-	const long want = (long)device_info().sms * (kBlockThreads / 32) * 2;
-	int R = (a.d + 3) / 4 >= want ? 4 : (a.d + 1) / 2 >= want ? 2 : 1; // rows per warp: 4 when that still gives every resident warp a task
+	// Rows per warp.  IN: two (four leave every CTA fewer, longer turns behind its staging: 10 % slower per token at widths 2048 and 4096).
+	// OUT stages long inputs, so fewer CTAs with two rows per warp when that still gives 12 warps per SM a task, else one.
+	int R = IN || (a.d + 1) / 2 >= (long)device_info().sms * 12 ? 2 : 1;
 	while (R < 4 && a.n / ch < 16 / R) R *= 2;                         // short rows: the 16 loads in flight must come from more rows
 	cudaError_t err = cudaSuccess;
 #define BLOCK_LAUNCH(DT_, R_)                                                                                                              \

@@ -108,20 +108,19 @@ __global__ void __launch_bounds__(128) conv_state_rows_kernel(const float *__res
 //   M <- a * M       (the decay a: one number per head, or one per head and key channel, acting on rows)
 //   e = beta * (v - M^T k)   (delta rule)   or   e = vscale * v
 //   M <- M + k e^T;   y = M^T q  (+ skip * v)
-// One CTA owns 16 columns of one head; 8 neighbouring lanes share a column, lane `sub` holding the EPL consecutive rows
-// sub * EPL .. in registers, so the two dot products of a step are EPL multiply-adds (four partial sums) and three shuffles.
+// One CTA owns 16 columns of one head; LPC neighbouring lanes (8 or 16) share LPC / 8 columns, lane `sub` holding the EPL consecutive
+// rows sub * EPL .. of each in registers, so a dot product of a step is EPL multiply-adds (four partial sums) and three or four shuffles.
 // k, q, the decays and v of 8 positions at a time go global -> shared with cp.async into one of two stages: the next 8 load
-// while these are consumed.  In shared memory a position's row is cut into the 8 lanes' segments, padded so that the lanes'
-// 16-byte reads fall into different banks.  The reduction of a position's output is carried into the next position's step,
-// where it shares the shuffle rounds of that step's M^T k, so only the recurrence itself (decay, M^T k, update) is a serial
-// chain.  The order of every sum is fixed, so a position's output does not depend on how the rows were cut into calls.
+// while these are consumed.  In shared memory a position's row is cut into the lanes' segments, padded so that the lanes'
+// 16-byte reads fall into different banks.  The outputs of a stage's 8 positions are reduced together at its end (LPC values,
+// position x column, over the LPC lanes by halving exchanges, one sum per lane), so only the recurrence itself (decay, M^T k, update) is
+// a serial chain.  The order of every sum is fixed, so a position's output does not depend on how the rows were cut into calls.
 // State in global memory: (head, column, row) fp32.
 struct ScanArgs {
 	float *out;
 	int ldo;
 	const float *k, *q, *v, *decay, *vscale, *beta, *skip;
 	int ldk, ldq, ldv, ldd, ldvs, ldb;
-	int decay_per_channel;
 	float *state;
 	int n, H, rep, D, P, pos0;
 	const int *ctl;
@@ -137,10 +136,10 @@ __device__ __forceinline__ void cp_async16f(float *smem, const float *gmem) {
 	asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(smem)), "l"(gmem) : "memory");
 }
 
-template <int EPL>
+template <int EPL, int LPC>
 struct ScanLayout {
 	static constexpr int SEG = EPL + (EPL >= 8 ? 4 : 0); // floats between two lanes' segments of a row
-	static constexpr int DP = 8 * SEG;
+	static constexpr int DP = LPC * SEG;
 	static constexpr int STAGE = 3 * kScanTok * DP + kScanTok * kScanCols + kScanTok * 4; // k, q, decay rows; v; (decay, vscale, beta) per position
 };
 
@@ -160,19 +159,27 @@ __device__ __forceinline__ void load_seg(float (&r)[EPL], const float *p) {
 		r[0] = p[0];
 }
 
-template <int EPL, bool BONUS>
+// MODE: kScanPerChannel, kScanDelta, kScanBonus or'ed (compile-time: a position's step is then free of branches and the unrolled
+// positions overlap).
+constexpr int kScanPerChannel = 1, kScanDelta = 2, kScanBonus = 4;
+template <int EPL, int MODE, int LPC>
 __global__ void __launch_bounds__(kScanCols * 8) state_scan_kernel(ScanArgs a) {
-	using LO = ScanLayout<EPL>;
+	constexpr bool BONUS = MODE & kScanBonus, DELTA = MODE & kScanDelta, PER_CHANNEL = MODE & kScanPerChannel;
+	using LO = ScanLayout<EPL, LPC>;
+	constexpr int NC = LPC / 8, GROUPS = kScanCols / NC; // columns per thread; column c0 + col + i GROUPS
 	constexpr int SEG = LO::SEG, DP = LO::DP, TOK = kScanTok, STAGE = LO::STAGE;
 	extern __shared__ __align__(16) float scan_sm[];
 	const int h = blockIdx.y, kh = h / a.rep, c0 = blockIdx.x * kScanCols;
-	const int tid = threadIdx.x, col = tid >> 3, sub = tid & 7;
-	const bool live = c0 + col < a.P;
+	const int tid = threadIdx.x, col = tid / LPC, sub = tid % LPC;
 	const bool fresh = first_pos(a.ctl, a.pos0) == 0;
-	float *sp = a.state + ((size_t)h * a.P + min(c0 + col, a.P - 1)) * a.D + sub * EPL;
-	float s[EPL];
+	auto state_at = [&](int i) { return a.state + ((size_t)h * a.P + min(c0 + col + i * GROUPS, a.P - 1)) * a.D + sub * EPL; };
+	float s[NC][EPL];
 #pragma unroll
-	for (int e = 0; e < EPL; ++e) s[e] = (!fresh && sub * EPL + e < a.D) ? sp[e] : 0.f;
+	for (int i = 0; i < NC; ++i) {
+		const float *sp = state_at(i);
+#pragma unroll
+		for (int e = 0; e < EPL; ++e) s[i][e] = (!fresh && sub * EPL + e < a.D) ? sp[e] : 0.f;
+	}
 	const float skip = a.skip ? a.skip[h] : 0.f;
 	float bu[BONUS ? EPL : 1];
 	if constexpr (BONUS)
@@ -193,14 +200,14 @@ __global__ void __launch_bounds__(kScanCols * 8) state_scan_kernel(ScanArgs a) {
 				const int t = idx / D4, i = (idx % D4) * 4, at = t * DP + (i / EPL) * SEG + i % EPL;
 				cp_async16f(ks + at, a.k + (size_t)(t0 + t) * a.ldk + kh * a.D + i);
 				cp_async16f(qs + at, a.q + (size_t)(t0 + t) * a.ldq + kh * a.D + i);
-				if (a.decay_per_channel) cp_async16f(gs + at, a.decay + (size_t)(t0 + t) * a.ldd + h * a.D + i);
+				if (PER_CHANNEL) cp_async16f(gs + at, a.decay + (size_t)(t0 + t) * a.ldd + h * a.D + i);
 			}
 		} else {
 			for (int idx = tid; idx < tc * a.D; idx += blockDim.x) {
 				const int t = idx / a.D, i = idx % a.D, at = t * DP + (i / EPL) * SEG + i % EPL;
 				cp_async4(ks + at, a.k + (size_t)(t0 + t) * a.ldk + kh * a.D + i);
 				cp_async4(qs + at, a.q + (size_t)(t0 + t) * a.ldq + kh * a.D + i);
-				if (a.decay_per_channel) cp_async4(gs + at, a.decay + (size_t)(t0 + t) * a.ldd + h * a.D + i);
+				if (PER_CHANNEL) cp_async4(gs + at, a.decay + (size_t)(t0 + t) * a.ldd + h * a.D + i);
 			}
 		}
 		for (int idx = tid; idx < tc * kScanCols; idx += blockDim.x) {
@@ -208,14 +215,78 @@ __global__ void __launch_bounds__(kScanCols * 8) state_scan_kernel(ScanArgs a) {
 			if (c0 + c < a.P) cp_async4(vs + idx, a.v + (size_t)(t0 + t) * a.ldv + h * a.P + c0 + c);
 		}
 		if (tid < tc) {
-			if (!a.decay_per_channel) cp_async4(sc + tid * 4, a.decay + (size_t)(t0 + tid) * a.ldd + h);
+			if (!PER_CHANNEL) cp_async4(sc + tid * 4, a.decay + (size_t)(t0 + tid) * a.ldd + h);
 			if (a.vscale) cp_async4(sc + tid * 4 + 1, a.vscale + (size_t)(t0 + tid) * a.ldvs + h);
-			if (a.beta) cp_async4(sc + tid * 4 + 2, a.beta + (size_t)(t0 + tid) * a.ldb + h);
+			if (DELTA) cp_async4(sc + tid * 4 + 2, a.beta + (size_t)(t0 + tid) * a.ldb + h);
 		}
 		asm volatile("cp.async.commit_group;" ::: "memory");
 	};
-	float po = 0.f, pvv = 0.f; // the previous position's output: partial sum of this lane, and its v
-	float *pout = nullptr;
+	// one position: the state moves on; what comes back is this lane's part of its columns' outputs
+	auto step = [&](float (&po)[NC], const float *ks, const float *qs, const float *gs, const float *vs, const float *sc, int t) {
+		float kt[EPL], qt[EPL];
+		load_seg<EPL>(kt, ks + t * DP + sub * SEG);
+		load_seg<EPL>(qt, qs + t * DP + sub * SEG);
+		float vv[NC], o4[NC][4];
+#pragma unroll
+		for (int i = 0; i < NC; ++i) {
+			vv[i] = vs[t * kScanCols + col + i * GROUPS];
+			o4[i][0] = o4[i][1] = o4[i][2] = o4[i][3] = 0.f;
+		}
+		if constexpr (BONUS) { // read-out of the state as it was, then decay and update
+			float gt[EPL];
+			load_seg<EPL>(gt, gs + t * DP + sub * SEG);
+#pragma unroll
+			for (int i = 0; i < NC; ++i)
+#pragma unroll
+				for (int e = 0; e < EPL; ++e) {
+					const float kv = kt[e] * vv[i];
+					o4[i][e & 3] = fmaf(fmaf(bu[e], kv, s[i][e]), qt[e], o4[i][e & 3]);
+					s[i][e] = fmaf(gt[e], s[i][e], kv);
+				}
+		} else {
+			if constexpr (PER_CHANNEL) {
+				float gt[EPL];
+				load_seg<EPL>(gt, gs + t * DP + sub * SEG);
+#pragma unroll
+				for (int i = 0; i < NC; ++i)
+#pragma unroll
+					for (int e = 0; e < EPL; ++e) s[i][e] *= gt[e];
+			} else {
+				const float d = sc[t * 4];
+#pragma unroll
+				for (int i = 0; i < NC; ++i)
+#pragma unroll
+					for (int e = 0; e < EPL; ++e) s[i][e] *= d;
+			}
+			float u[NC];
+			if constexpr (DELTA) {
+#pragma unroll
+				for (int i = 0; i < NC; ++i) {
+					float d4[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+					for (int e = 0; e < EPL; ++e) d4[e & 3] = fmaf(s[i][e], kt[e], d4[e & 3]);
+					u[i] = (d4[0] + d4[1]) + (d4[2] + d4[3]);
+				}
+#pragma unroll
+				for (int o = LPC / 2; o > 0; o >>= 1)
+#pragma unroll
+					for (int i = 0; i < NC; ++i) u[i] += __shfl_xor_sync(kFull, u[i], o);
+#pragma unroll
+				for (int i = 0; i < NC; ++i) u[i] = sc[t * 4 + 2] * (vv[i] - u[i]);
+			} else
+#pragma unroll
+				for (int i = 0; i < NC; ++i) u[i] = sc[t * 4 + 1] * vv[i];
+#pragma unroll
+			for (int i = 0; i < NC; ++i)
+#pragma unroll
+				for (int e = 0; e < EPL; ++e) {
+					s[i][e] = fmaf(kt[e], u[i], s[i][e]);
+					o4[i][e & 3] = fmaf(s[i][e], qt[e], o4[i][e & 3]);
+				}
+		}
+#pragma unroll
+		for (int i = 0; i < NC; ++i) po[i] = (o4[i][0] + o4[i][1]) + (o4[i][2] + o4[i][3]);
+	};
 	issue(0, 0);
 	for (int c = 0, t0 = 0; t0 < a.n; ++c, t0 += TOK) {
 		const int tc = min(TOK, a.n - t0);
@@ -226,70 +297,39 @@ __global__ void __launch_bounds__(kScanCols * 8) state_scan_kernel(ScanArgs a) {
 			asm volatile("cp.async.wait_group 0;" ::: "memory");
 		__syncthreads();
 		const float *ks = scan_sm + (c & 1) * STAGE, *qs = ks + TOK * DP, *gs = qs + TOK * DP, *vs = gs + TOK * DP, *sc = vs + TOK * kScanCols;
-		for (int t = 0; t < tc; ++t) {
-			float kt[EPL], qt[EPL];
-			load_seg<EPL>(kt, ks + t * DP + sub * SEG);
-			load_seg<EPL>(qt, qs + t * DP + sub * SEG);
-			const float vv = vs[t * kScanCols + col];
-			if constexpr (BONUS) { // read-out of the state as it was, then decay and update
-				float gt[EPL];
-				load_seg<EPL>(gt, gs + t * DP + sub * SEG);
-				po += __shfl_xor_sync(kFull, po, 4), po += __shfl_xor_sync(kFull, po, 2), po += __shfl_xor_sync(kFull, po, 1);
-				if (pout && sub == 0 && live) *pout = po;
-				float o4[4] = {0.f, 0.f, 0.f, 0.f};
+		float po[TOK][NC];
+		if (tc == TOK) { // unrolled: the next positions' operands are read while a position's chain waits
 #pragma unroll
-				for (int e = 0; e < EPL; ++e) {
-					const float kv = kt[e] * vv;
-					o4[e & 3] = fmaf(fmaf(bu[e], kv, s[e]), qt[e], o4[e & 3]);
-					s[e] = fmaf(gt[e], s[e], kv);
-				}
-				po = (o4[0] + o4[1]) + (o4[2] + o4[3]);
-				pout = a.out + (size_t)(t0 + t) * a.ldo + h * a.P + min(c0 + col, a.P - 1);
-				continue;
+			for (int t = 0; t < TOK; ++t) step(po[t], ks, qs, gs, vs, sc, t);
+		} else {
+#pragma unroll
+			for (int t = 0; t < TOK; ++t) {
+#pragma unroll
+				for (int i = 0; i < NC; ++i) po[t][i] = 0.f;
+				if (t < tc) step(po[t], ks, qs, gs, vs, sc, t);
 			}
-			if (a.decay_per_channel) {
-				float gt[EPL];
-				load_seg<EPL>(gt, gs + t * DP + sub * SEG);
-#pragma unroll
-				for (int e = 0; e < EPL; ++e) s[e] *= gt[e];
-			} else {
-				const float d = sc[t * 4];
-#pragma unroll
-				for (int e = 0; e < EPL; ++e) s[e] *= d;
-			}
-			float u;
-			if (a.beta) {
-				float d4[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll
-				for (int e = 0; e < EPL; ++e) d4[e & 3] = fmaf(s[e], kt[e], d4[e & 3]);
-				float dot = (d4[0] + d4[1]) + (d4[2] + d4[3]);
-				dot += __shfl_xor_sync(kFull, dot, 4), po += __shfl_xor_sync(kFull, po, 4);
-				dot += __shfl_xor_sync(kFull, dot, 2), po += __shfl_xor_sync(kFull, po, 2);
-				dot += __shfl_xor_sync(kFull, dot, 1), po += __shfl_xor_sync(kFull, po, 1);
-				u = sc[t * 4 + 2] * (vv - dot);
-			} else {
-				po += __shfl_xor_sync(kFull, po, 4), po += __shfl_xor_sync(kFull, po, 2), po += __shfl_xor_sync(kFull, po, 1);
-				u = sc[t * 4 + 1] * vv;
-			}
-			if (pout && sub == 0 && live) *pout = po + skip * pvv;
-			float o4[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll
-			for (int e = 0; e < EPL; ++e) {
-				s[e] = fmaf(kt[e], u, s[e]);
-				o4[e & 3] = fmaf(s[e], qt[e], o4[e & 3]);
-			}
-			po = (o4[0] + o4[1]) + (o4[2] + o4[3]), pvv = vv;
-			pout = a.out + (size_t)(t0 + t) * a.ldo + h * a.P + min(c0 + col, a.P - 1);
 		}
+		// the LPC values (position, column) of the stage over the column's LPC lanes: halving exchanges leave lane `sub` with the sum of value `sub`
+		float *pv = &po[0][0];
+#pragma unroll
+		for (int o = LPC / 2; o > 0; o >>= 1)
+#pragma unroll
+			for (int i = 0; i < o; ++i) {
+				const float give = (sub & o) ? pv[i] : pv[i + o], keep = (sub & o) ? pv[i + o] : pv[i];
+				pv[i] = keep + __shfl_xor_sync(kFull, give, o);
+			}
+		const int ot = sub / NC, oc = col + (sub % NC) * GROUPS;
+		if (c0 + oc < a.P && ot < tc) a.out[(size_t)(t0 + ot) * a.ldo + h * a.P + c0 + oc] = pv[0] + skip * vs[ot * kScanCols + oc];
 		__syncthreads(); // this stage is consumed: the copies of the position group after next may land in it
 	}
-	po += __shfl_xor_sync(kFull, po, 4), po += __shfl_xor_sync(kFull, po, 2), po += __shfl_xor_sync(kFull, po, 1);
-	if (pout && sub == 0 && live) *pout = po + skip * pvv;
-	if (live) {
 #pragma unroll
-		for (int e = 0; e < EPL; ++e)
-			if (sub * EPL + e < a.D) sp[e] = s[e];
-	}
+	for (int i = 0; i < NC; ++i)
+		if (c0 + col + i * GROUPS < a.P) {
+			float *sp = state_at(i);
+#pragma unroll
+			for (int e = 0; e < EPL; ++e)
+				if (sub * EPL + e < a.D) sp[e] = s[i][e];
+		}
 }
 
 // dt[m, h] = softplus(dt + bias[h]) in place; decay[m, h] = exp(-exp(a_log[h]) * dt)
@@ -656,24 +696,27 @@ extern "C" int yalm_conv_act_rows(float *out, int ldo, const float *in, int ldi,
 	return (int)cudaGetLastError();
 }
 
-template <bool BONUS>
+template <int MODE>
 static int launch_scan(const ScanArgs &a, dim3 grid, cudaStream_t st) {
-#define SCAN_CASE(EPL_)                                                                                                                      \
+#define SCAN_CASE(EPL_, LPC_)                                                                                                                \
 	{                                                                                                                                        \
-		constexpr size_t smem = sizeof(float) * 2 * ScanLayout<EPL_>::STAGE;                                                                 \
+		constexpr size_t smem = sizeof(float) * 2 * ScanLayout<EPL_, LPC_>::STAGE;                                                           \
 		static bool configured = false;                                                                                                      \
 		if (smem > 48 * 1024 && !configured) {                                                                                               \
-			YALM_TRY(cudaFuncSetAttribute(state_scan_kernel<EPL_, BONUS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));          \
+			YALM_TRY(cudaFuncSetAttribute(state_scan_kernel<EPL_, MODE, LPC_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));     \
 			configured = true;                                                                                                               \
 		}                                                                                                                                    \
-		state_scan_kernel<EPL_, BONUS><<<grid, kScanCols * 8, smem, st>>>(a);                                                                \
+		state_scan_kernel<EPL_, MODE, LPC_><<<grid, kScanCols * 8, smem, st>>>(a);                                                           \
 	}
-	if (a.D <= 8) SCAN_CASE(1)
-	else if (a.D <= 16) SCAN_CASE(2)
-	else if (a.D <= 32) SCAN_CASE(4)
-	else if (a.D <= 64) SCAN_CASE(8)
-	else if (a.D <= 128) SCAN_CASE(16)
-	else SCAN_CASE(32)
+	// lanes per column: the delta rule's chain through the shuffles is shortest with 8; without it, two columns per thread on 16 lanes read
+	// each operand from shared memory half as often (D = 64, 512 rows of 32 heads: 74 -> 62 us; delta rule 96 -> 104 us)
+	constexpr bool wide = !(MODE & kScanDelta);
+	if (a.D <= 8) SCAN_CASE(1, 8)
+	else if (a.D <= 16) SCAN_CASE(2, 8)
+	else if (a.D <= 32) SCAN_CASE(4, 8)
+	else if (a.D <= 64) SCAN_CASE(wide ? 4 : 8, wide ? 16 : 8)
+	else if (a.D <= 128) SCAN_CASE(wide ? 8 : 16, wide ? 16 : 8)
+	else SCAN_CASE(wide ? 16 : 32, wide ? 16 : 8)
 #undef SCAN_CASE
 	return (int)cudaGetLastError();
 }
@@ -686,9 +729,11 @@ extern "C" int yalm_state_scan_rows(float *out, int ldo, const float *k, int ldk
 	if (!out || !k || !q || !v || !decay || !state || n < 1 || heads < 1 || rep < 1 || heads % rep || D < 1 || D > kScanMaxD || P < 1) return YALM_EINVAL;
 	auto al = [](const float *p, int ld) { return ((uintptr_t)p & 15) == 0 && ld % 4 == 0; };
 	const int vec = D % 4 == 0 && al(k, ldk) && al(q, ldq) && (!decay_per_channel || al(decay, ldd));
-	ScanArgs a{out, ldo, k, q, v, decay, vscale, beta, skip, ldk, ldq, ldv, ldd, ldvs, ldb, decay_per_channel, state, n, heads, rep, D, P, pos0, ctl, vec};
+	ScanArgs a{out, ldo, k, q, v, decay, vscale, beta, skip, ldk, ldq, ldv, ldd, ldvs, ldb, state, n, heads, rep, D, P, pos0, ctl, vec};
 	const dim3 grid((P + kScanCols - 1) / kScanCols, heads);
-	return launch_scan<false>(a, grid, (cudaStream_t)s);
+	cudaStream_t st = (cudaStream_t)s;
+	if (beta) return decay_per_channel ? launch_scan<kScanDelta | kScanPerChannel>(a, grid, st) : launch_scan<kScanDelta>(a, grid, st);
+	return decay_per_channel ? launch_scan<kScanPerChannel>(a, grid, st) : launch_scan<0>(a, grid, st);
 }
 
 // The time-mixing recurrence: out = (M + diag(bonus) k v^T)^T q, M <- decay M + k v^T; k, q, decay (n, H D), v, out (n, H P), bonus (H, D).
@@ -696,9 +741,9 @@ extern "C" int yalm_state_scan_bonus_rows(float *out, int ldo, const float *k, i
                                           int ldd, const float *bonus, float *state, int n, int heads, int D, int P, int pos0, const int *ctl, yalm_stream_t s) {
 	if (!out || !k || !q || !v || !decay || !bonus || !state || n < 1 || heads < 1 || D < 1 || D > kScanMaxD || P < 1) return YALM_EINVAL;
 	auto al = [](const float *p, int ld) { return ((uintptr_t)p & 15) == 0 && ld % 4 == 0; };
-	ScanArgs a{out, ldo, k, q, v, decay, nullptr, nullptr, nullptr, ldk, ldq, ldv, ldd, 0, 0, 1, state, n, heads, 1, D, P, pos0, ctl,
+	ScanArgs a{out, ldo, k, q, v, decay, nullptr, nullptr, nullptr, ldk, ldq, ldv, ldd, 0, 0, state, n, heads, 1, D, P, pos0, ctl,
 	           D % 4 == 0 && al(k, ldk) && al(q, ldq) && al(decay, ldd), bonus};
-	return launch_scan<true>(a, dim3((P + kScanCols - 1) / kScanCols, heads), (cudaStream_t)s);
+	return launch_scan<kScanBonus | kScanPerChannel>(a, dim3((P + kScanCols - 1) / kScanCols, heads), (cudaStream_t)s);
 }
 
 extern "C" int yalm_ssm_prep_rows(float *dt, int lddt, float *decay, int ldd, const float *dt_bias, const float *a_log, int n, int heads, yalm_stream_t s) {
