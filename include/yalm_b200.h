@@ -633,6 +633,48 @@ int yalm_gemv_block_out(float *res, const float *x1, int n1, const float *gu, in
 int yalm_gemm_16_segments(float *c, int ldc, const void *a, const void *w, int M, int N, int K, int n_segments, const int *segment_end, int bf16,
                           yalm_stream_t s);
 
+/* ---- attention whose heads exchange scores, retention, norms in groups (csrc/ops_stack_talk.cu, ops_stack_block.cu) ----
+ * out[i, h] = sum_j a_h(j) v(j) (times sigmoid(gate[i, h]); gate NULL: not), a_h the softmax over 0 <= i - j < window (0: all j <= i) of
+ * sum_g mix[h, g] (cap tanh(q_g . k(j) scale / cap) + bias[g, min(i - j, n_bias - 1)]); softcap 0: no cap, bias NULL: none, mix NULL: own
+ * score only.  q (n, n_heads dk), key / value rings (n_kv, ring, dk | dv), bias (n_heads, n_bias), mix (n_heads, n_heads), gate row stride ldg.
+ * workspace: split partials, yalm_attn_mixed_workspace floats (fewer: fewer splits), or NULL.  _rows: any sizes, fp32 or bf16 rings;
+ * _decode / _mma: bf16 rings on the tensor cores, for few rows / prompt portions, when the _shape function returns a key tile (0: no
+ * kernel); q and the rings 16-byte aligned, ldq a multiple of 4. */
+size_t yalm_attn_mixed_workspace(int rows, int heads, int dv);
+int yalm_attn_mixed_rows(float *out, int ldo, const float *q, int ldq, const void *key_ring, const void *value_ring, const float *bias, int n_bias,
+                         const float *mix, const float *gate, int ldg, float *workspace, size_t workspace_floats, int n, int n_heads, int n_kv, int dk,
+                         int dv, int ring, int window, float scale, float softcap, int cache_f32, int context, int pos0, const int *ctl, yalm_stream_t s);
+int yalm_attn_mixed_decode_shape(int n_heads, int n_kv, int dk, int dv);
+int yalm_attn_mixed_decode(float *out, int ldo, const float *q, int ldq, const void *key_ring, const void *value_ring, const float *bias, int n_bias,
+                           const float *mix, const float *gate, int ldg, float *workspace, size_t workspace_floats, int n, int n_heads, int n_kv, int dk,
+                           int dv, int ring, int window, float scale, float softcap, int context, int pos0, const int *ctl, yalm_stream_t s);
+int yalm_attn_mixed_mma_shape(int n_heads, int n_kv, int dk, int dv);
+int yalm_attn_mixed_mma(float *out, int ldo, const float *q, int ldq, const void *key_ring, const void *value_ring, const float *bias, int n_bias,
+                        const float *mix, const float *gate, int ldg, float *workspace, size_t workspace_floats, int n, int n_heads, int n_kv, int dk, int dv,
+                        int ring, int window, float scale, float softcap, int context, int pos0, const int *ctl, yalm_stream_t s);
+/* yalm_attn_latent_merge with, optionally, every head's result times sigmoid(gate[row, head]). */
+int yalm_attn_split_merge(float *out, int ldo, const float *part, int n, int n_heads, int dv, int nsplit, const float *sink, const float *gate, int ldg,
+                          yalm_stream_t s);
+/* yalm_qkv_post_rows with biases (q | k | v; NULL: none) added first. */
+int yalm_qkv_bias_post_rows(float *qkv, int ld, const float *bias, void *key_ring, void *value_ring, float *vfirst, int ldvf, const float *qnorm,
+                            const float *knorm, const float *vmix, int vmode, int n, int n_heads, int n_kv, int dk, int dv, int ring, float eps,
+                            int cache_f32, int pos0, const int *ctl, yalm_stream_t s);
+/* A decode row of retention in one launch: q and k rotated, M <- decay[h] M + k_scale k v^T, o = M^T q, out = o / sqrt(mean o^2 + eps) per head
+ * times silu(gate).  proj: the row of the packed projection (o_*: offsets); state (heads, vdim, dim) fp32.  dim <= 256. */
+int yalm_retention_step(float *out, float *state, const float *proj, int o_q, int o_k, int o_v, int o_gate, const float *decay, const float *freq,
+                        float magnitude, int rot_dims, int interleaved, float k_scale, int heads, int dim, int vdim, float eps, int pos0, const int *ctl,
+                        yalm_stream_t s);
+/* out[r] and / or out16[r] = row rows[r] (NULL: r) of x, each of `groups` equal parts over its own root mean square, times w (dim). */
+int yalm_group_norm_rows(float *out, void *out16, int bf16, const float *x, const int *rows, const float *w, int groups, float eps, int n, int dim,
+                         yalm_stream_t s);
+/* x += mult * (a + a_bias + b + sum_j y_j) (y: nsum rows of stride ldy per row of x; NULL: left out), then the same norm of x (w NULL: none). */
+int yalm_residual_group_norm_rows(float *x, float mult, const float *a, const float *a_bias, const float *b, const float *y, int ldy, int nsum, float *out,
+                                  void *out16, int bf16, const float *w, int groups, float eps, int n, int dim, yalm_stream_t s);
+/* yalm_router_bias_topk_rows where a group is ranked by the sum of its group_top best experts' choice scores (1: by the best). */
+int yalm_router_group_topk_rows(int *ids, float *wts, const float *x, int ldx, const void *wr, int dtype, int n, int n_experts, int top, int dim, int score,
+                                int renorm, float renorm_eps, int groups, int keep_groups, int group_top, const float *bias, float weight_scale,
+                                yalm_stream_t s);
+
 #ifdef __cplusplus
 }
 #endif

@@ -48,6 +48,8 @@ SYMBOLS = [
     "yalm_embed_bigram_rows", "yalm_layer_norm_rows", "yalm_mix_rows", "yalm_delta_in_rows", "yalm_wkv_decay_rows", "yalm_state_scan_bonus_rows",
     "yalm_head_bias_rope_norm_append_rows", "yalm_block_out_rows", "yalm_delta_step", "yalm_wkv_step", "yalm_gemv_block_in", "yalm_gemv_block_out",
     "yalm_gemm_16_segments",
+    "yalm_attn_mixed_workspace", "yalm_attn_mixed_rows", "yalm_attn_mixed_decode_shape", "yalm_attn_mixed_decode", "yalm_attn_mixed_mma_shape", "yalm_attn_mixed_mma",
+    "yalm_attn_split_merge", "yalm_qkv_bias_post_rows", "yalm_retention_step", "yalm_group_norm_rows", "yalm_residual_group_norm_rows", "yalm_router_group_topk_rows",
     "yalm_tp_unique_id", "yalm_tp_init", "yalm_tp_finalize", "yalm_tp_shard_plan", "yalm_mega_tile_plan", "yalm_mega_attn_split", "yalm_mega_mma_plan", "yalm_mega_hb_share", "yalm_error_string", "yalm_version",
 ]
 

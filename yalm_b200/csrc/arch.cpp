@@ -153,7 +153,7 @@ int StackSpec::max_v_dim() const {
 int StackSpec::max_o_dim() const {
 	int m = 0;
 	for (const LayerSpec &l : layers)
-		m = std::max({m, l.mix.heads * l.mix.maps * l.mix.vdim, l.ssm.inner(), l.delta.heads * l.delta.vdim, l.mix.heads * l.latent.kv_rank, l.gla.heads * l.gla.vdim, l.wkv.inner()});
+		m = std::max({m, l.mix.heads * l.mix.maps * l.mix.vdim, l.ssm.inner(), l.delta.heads * l.delta.vdim, l.mix.heads * l.latent.kv_rank, l.gla.heads * l.gla.vdim, l.wkv.inner(), l.ret.heads * l.ret.vdim});
 	return m;
 }
 int StackSpec::max_block_out() const {
@@ -193,6 +193,9 @@ int LayerSpec::proj_width() const {
 	if (kind == MixerKind::LatentAttention) // [query latent, or the queries themselves | key / value latent + shared key part (own cache only) | gate]
 		return (latent.q_rank > 0 ? latent.q_rank : mix.heads * (mix.dim + latent.rot_dim)) + (latent.kv_from < 0 ? latent.kv_rank + latent.rot_dim : 0) +
 		       (mix.out_gate ? mix.heads * mix.vdim : 0);
+	if (kind == MixerKind::Retention) return (2 * ret.heads * (ret.dim + ret.vdim) + 7) & ~7; // [q | k | v | gate]
+	if (kind == MixerKind::Attention && mix.talk) // [q | k | v | one gate per head]
+		return ((mix.heads + mix.kv_heads) * mix.dim + mix.kv_heads * mix.vdim + (mix.head_gate ? mix.heads : 0) + 7) & ~7;
 	if (kind == MixerKind::LinearAttention) return 2 * gla.heads * gla.dim + 2 * gla.heads * gla.vdim + gla.decay_rank;
 	// packed blocks (rows padded to a multiple of 8): the mixer's large projections, the feed-forward's gate and up, then what is not
 	// a multiple of anything
@@ -210,6 +213,7 @@ int LayerSpec::mixed_width() const {
 	if (kind == MixerKind::LinearAttention) return gla.heads * gla.vdim;
 	if (kind == MixerKind::DeltaRule) return delta.heads * delta.vdim;
 	if (kind == MixerKind::TimeMix) return wkv.inner();
+	if (kind == MixerKind::Retention) return ret.heads * ret.vdim;
 	return mix.heads * mix.vdim + (kind == MixerKind::Parallel ? delta.heads * delta.vdim : 0);
 }
 int LayerSpec::conv_width() const {
@@ -1002,12 +1006,168 @@ int configure_fafelix(const JValue &j, Config &cfg) {
 	return 0;
 }
 
+// ---- Desalorn --------------------------------------------------------------------------------------------------------
+// A decoder-only stack of parallel blocks, x <- x + m (mixer(h) + experts(h)) with ONE norm h = N(x) per layer, an RMS norm of equal
+// parts of the vector.  Mixers: attention without rotation (biased projections, RMS norm over the whole q and k, soft-capped scores plus
+// a learned distance bias, the heads' scores mixed by a stored matrix, one sigmoid gate number per head); retention (rotary q and k,
+// a matrix state per head with a fixed decay, per-head norm without a weight, SiLU gate); latent attention over a window of cached
+// latents.  Experts: sigmoid router whose choice adds a stored correction, restricted to the groups with the best two experts, raw
+// scores as weights; a shared expert beside them.
+std::string desalorn_tensor(int layer, TensorRole role, int expert) {
+	const std::string l = "l" + std::to_string(layer) + ".", m = l + "mix.", f = l + "mlp.";
+	const std::string e = expert >= 0 ? f + "e" + std::to_string(expert) + "." : f;
+	switch (role) {
+	case TensorRole::Embed: return "embed";
+	case TensorRole::FinalNorm: return "final.norm";
+	case TensorRole::Head: return "head";
+	case TensorRole::Norm1: return l + "norm1";
+	case TensorRole::Wq: return m + "q";
+	case TensorRole::Wk: return m + "k";
+	case TensorRole::Wv: return m + "v";
+	case TensorRole::Wo: return m + "o";
+	case TensorRole::QBias: return m + "q.b";
+	case TensorRole::KBias: return m + "k.b";
+	case TensorRole::VBias: return m + "v.b";
+	case TensorRole::WoBias: return m + "o.b";
+	case TensorRole::QNorm: return m + "q.norm";
+	case TensorRole::KNorm: return m + "k.norm";
+	case TensorRole::RelBias: return m + "rel";
+	case TensorRole::Talk: return m + "talk";
+	case TensorRole::OutGate: return m + "g";
+	case TensorRole::LatentDq: return m + "dq";
+	case TensorRole::LatentDqNorm: return m + "dq.norm";
+	case TensorRole::LatentUq: return m + "uq";
+	case TensorRole::LatentDkv: return m + "dkv";
+	case TensorRole::LatentDkvNorm: return m + "dkv.norm";
+	case TensorRole::LatentUk: return m + "uk";
+	case TensorRole::LatentUv: return m + "uv";
+	case TensorRole::Router: return f + "router";
+	case TensorRole::RouterBias: return f + "correction";
+	case TensorRole::Gate: return e + "gate";
+	case TensorRole::Up: return e + "up";
+	case TensorRole::Down: return e + "down";
+	case TensorRole::SharedGate: return f + "shared.gate";
+	case TensorRole::SharedUp: return f + "shared.up";
+	case TensorRole::SharedDown: return f + "shared.down";
+	default: break;
+	}
+	return "";
+}
+
+int fail_desalorn(const char *what) {
+	fprintf(stderr, "yalm_b200: Desalorn config.json: %s\n", what);
+	return YALM_EFORMAT;
+}
+
+// No table bounds the context: the key / value rings of the unbounded attention layers are sized by the context the caller asks for,
+// else by "max_positions", else by this.
+constexpr int kDesalornContext = 32768;
+
+int configure_desalorn(const JValue &j, Config &cfg) {
+	auto spec = std::make_shared<StackSpec>();
+	StackSpec &s = *spec;
+	s.arch = "Desalorn";
+	s.width = j["width"].integer(0);
+	s.vocab = j["vocab"].integer(0);
+	s.max_positions = j["max_positions"].integer(kDesalornContext);
+	s.norm_eps = (float)j["norm"]["eps"].number(1e-5);
+	s.norm_groups = j["norm"]["groups"].integer(1);
+	s.embed_scale = (float)j["embedding"]["scale"].number(1.0);
+	s.residual_mult = (float)j["residual_mult"].number(1.0);
+	s.parallel_block = true;
+	s.tensor_name = desalorn_tensor;
+	if (s.width < 1 || s.vocab < 1 || s.max_positions < 1) return fail_desalorn("width and vocab must be positive");
+	if (s.norm_groups < 1 || s.width % s.norm_groups) return fail_desalorn("norm.groups must divide the width");
+	const JValue &layers = j["layers"];
+	if (!layers.is_array() || layers.arr.empty()) return fail_desalorn("'layers' must be a non-empty list");
+	for (const JValue &jl : layers.arr) {
+		LayerSpec L;
+		const std::string type = jl["type"].string_or("");
+		const JValue &m = jl["mixer"];
+		MixerSpec &x = L.mix;
+		if (type == "attention") {
+			L.kind = MixerKind::Attention;
+			x.heads = m["heads"].integer(0), x.kv_heads = m["kv_heads"].integer(x.heads);
+			x.dim = m["dim"].integer(0), x.vdim = m["vdim"].integer(x.dim);
+			x.scale = (float)m["scale"].number(1.0);
+			x.softcap = (float)m["softcap"].number(0.0);
+			x.rel_rows = 1, x.rel_far = m["bias_max"].integer(0); // the table's shape gives the rows
+			x.qk_norm = QkNorm::WholeProjection;
+			x.talk = x.head_gate = x.qk_bias = x.v_bias = x.o_bias = true;
+			if (x.heads < 1 || x.kv_heads < 1 || x.heads % x.kv_heads || x.dim < 1 || x.vdim < 1 || !(x.softcap >= 0.f) || x.rel_far < 1)
+				return fail_desalorn("bad attention sizes");
+		} else if (type == "retention") {
+			L.kind = MixerKind::Retention;
+			RetentionSpec &r = L.ret;
+			r.heads = m["heads"].integer(0), r.dim = m["dim"].integer(0), r.vdim = m["vdim"].integer(r.dim);
+			r.rot.dims = m["rot"]["dims"].integer(r.dim), r.rot.base = m["rot"]["base"].number(10000.0), r.rot.interleaved = false;
+			const JValue &d = m["decay"];
+			if (d.is_array())
+				for (const JValue &v : d.arr) r.decay.push_back((float)v.number(0.0));
+			if (r.heads < 1 || r.dim < 1 || r.vdim < 1 || (int)r.decay.size() != r.heads) return fail_desalorn("bad retention sizes (decay: one number per head)");
+			if (r.rot.dims < 0 || r.rot.dims % 2 || r.rot.dims > r.dim || !(r.rot.base > 0.0)) return fail_desalorn("rot.dims must be even and at most dim");
+		} else if (type == "latent_attention") {
+			L.kind = MixerKind::LatentAttention;
+			LatentSpec &y = L.latent;
+			x.heads = m["heads"].integer(0), x.kv_heads = 1; // every head reads the one cached row of a position
+			x.dim = m["dim"].integer(0), x.vdim = m["vdim"].integer(0);
+			x.scale = (float)m["scale"].number(1.0);
+			x.window = m["mask"]["size"].integer(0);
+			y.q_rank = m["q_rank"].integer(0), y.kv_rank = m["kv_rank"].integer(0), y.rot_dim = m["rot_dim"].integer(0);
+			y.rot.dims = m["rot"]["dims"].integer(y.rot_dim), y.rot.base = m["rot"]["base"].number(10000.0), y.rot.interleaved = true;
+			if (x.heads < 1 || x.dim < 0 || x.vdim < 1 || x.window < 0 || y.q_rank < 1 || y.kv_rank < 1 || y.rot_dim < 0 || x.dim + y.rot_dim < 1)
+				return fail_desalorn("bad latent-attention sizes");
+			if (y.rot.dims < 0 || y.rot.dims % 2 || y.rot.dims > y.rot_dim || !(y.rot.base > 0.0)) return fail_desalorn("rot.dims must be even and at most rot_dim");
+		} else
+			return fail_desalorn("unknown layer type (this build has: attention, retention, latent_attention)");
+		const JValue &f = jl["mlp"];
+		if (f.is_object()) {
+			if (f["kind"].string_or("") != "moe") return fail_desalorn("unknown mlp kind (this build has: moe)");
+			FfnSpec &F = L.ffn;
+			const JValue &r = f["router"];
+			F.kind = FfnSpec::Moe, F.act = GluAct::Silu;
+			F.ff = f["expert"]["ff"].integer(0);
+			F.experts = r["experts"].integer(0), F.top = r["top"].integer(0);
+			F.score = RouterScore::Sigmoid, F.choice_bias = true;
+			if (r["groups"].is_object()) F.groups = r["groups"]["count"].integer(1), F.keep_groups = r["groups"]["keep"].integer(1);
+			F.group_top = 2;
+			if (f["shared"].is_object()) {
+				F.shared_ff = f["shared"]["ff"].integer(0), F.shared_act = GluAct::Silu;
+				if (F.shared_ff < 1) return fail_desalorn("bad shared expert size");
+			}
+			if (F.experts < 1 || F.experts > 1024 || F.ff < 1 || F.top < 1 || F.groups < 1 || F.experts % F.groups || F.keep_groups < 1 || F.keep_groups > F.groups ||
+			    F.top > F.keep_groups * (F.experts / F.groups))
+				return fail_desalorn("bad router sizes");
+		}
+		s.layers.push_back(L);
+	}
+	cfg.stack = spec;
+	cfg.dim = s.width;
+	cfg.vocab_size = s.vocab;
+	cfg.n_layers = (int)s.layers.size();
+	cfg.max_seq_len = s.max_positions;
+	cfg.norm_eps = s.norm_eps;
+	cfg.hidden_dim = std::max(1, s.max_ff());
+	cfg.n_heads = cfg.n_kv_heads = 1;
+	for (const LayerSpec &l : s.layers)
+		if (l.kind == MixerKind::Attention) {
+			cfg.n_heads = l.mix.heads, cfg.n_kv_heads = l.mix.kv_heads;
+			break;
+		}
+	cfg.head_dim = 8;
+	while (cfg.n_heads * cfg.head_dim < std::max({s.max_aux(), s.max_o_dim(), s.max_q_dim()})) cfg.head_dim *= 2;
+	cfg.rotary_dim = 0;
+	cfg.n_experts = s.max_experts(), cfg.n_experts_active = s.max_top();
+	return 0;
+}
+
 const ArchEntry kArchs[] = {
     {"Retezen", configure_retezen},
     {"Fapudra", configure_fapudra},
     {"Fegizen", configure_fegizen},
     {"Kiduvik", configure_kiduvik},
     {"Fafelix", configure_fafelix},
+    {"Desalorn", configure_desalorn},
 };
 
 } // namespace

@@ -40,7 +40,8 @@ enum class MixerKind {
 	LatentAttention, // MixerSpec + LatentSpec: queries, keys and values through low-rank latents; the cache holds the key / value latent
 	LinearAttention, // GlaSpec: a (dim, vdim) matrix state per head with one decay per key channel
 	DeltaRule,       // DeltaSpec alone
-	TimeMix          // WkvSpec: a matrix state with one decay per key channel, read out before the decay with a bonus for the current token
+	TimeMix,         // WkvSpec: a matrix state with one decay per key channel, read out before the decay with a bonus for the current token
+	Retention        // RetentionSpec: a (dim, vdim) matrix state per head with a fixed decay
 };
 // How attention scores become weights.
 enum class AttnWeights { Softmax, Sigmoid /* sigmoid(score + head bias), not normalised over the keys */ };
@@ -82,6 +83,9 @@ struct MixerSpec {
 	                             // values; per head o = a_1 - lambda a_2, o / sqrt(mean o^2 + eps) (1 - diff), with
 	float diff = 0.f;            // lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff from four stored vectors of size dim
 	bool head_gate = false;      // every head's output times sigmoid(w_h . input), one number per head, before the output projection
+	float softcap = 0.f;         // > 0: scaled scores pass softcap * tanh(score / softcap), before the distance bias
+	bool talk = false;           // the heads' scores are mixed by a stored (heads, heads) matrix, last thing before the softmax
+	bool o_bias = false;         // a bias on the output projection
 	bool sink = false;           // a stored number per head joins the softmax's denominator as exp(sink_h): no key, no value, not scaled
 };
 
@@ -139,6 +143,14 @@ struct WkvSpec {
 	int inner() const { return heads * dim; }
 };
 
+// Retention: q and k rotated, per head S <- decay_h S + k v^T with k scaled by dim^(-1/2), out = S^T q; per head out over its root mean
+// square (no weight), times silu(W_g x).
+struct RetentionSpec {
+	int heads = 0, dim = 0, vdim = 0;
+	RotarySpec rot;
+	std::vector<float> decay; // one per head
+};
+
 struct FfnSpec {
 	enum Kind { None, Dense, Moe } kind = None;
 	int ff = 0;                  // hidden size (per expert for Moe)
@@ -150,8 +162,8 @@ struct FfnSpec {
 	RouterScore score = RouterScore::Softmax;
 	bool renormalize = false;    // selected scores divided by their sum
 	float renorm_eps = 0.f;      // ... plus this
-	int groups = 1, keep_groups = 1; // experts form `groups` equal groups of neighbours; a group scores its best expert and only
-	                             // the keep_groups best groups' experts can be chosen
+	int groups = 1, keep_groups = 1; // experts form `groups` equal groups of neighbours; a group scores the sum of its group_top best experts
+	int group_top = 1;           // (choice scores) and only the keep_groups best groups' experts can be chosen
 	bool weight_on_input = false; // expert(w * h) instead of w * expert(h)
 	int identity = 0;            // the router has experts + identity outputs; the last `identity` stand for experts that return their input
 	bool choice_bias = false;    // experts are chosen by score + a stored bias per router output; the weights use the score alone
@@ -169,6 +181,7 @@ struct LayerSpec {
 	LatentSpec latent;
 	GlaSpec gla;
 	WkvSpec wkv;
+	RetentionSpec ret;
 	float left_scale = 1.f, right_scale = 1.f; // Parallel: left_scale * attention + right_scale * delta rule
 	FfnSpec ffn;
 	// widths of what the layer computes per row, for scratch sizing
@@ -203,7 +216,8 @@ enum class TensorRole {
 	GlaNorm, GlaDecay1, GlaDecay2, GlaDecayBias,
 	Norm1Post, Norm2Post, Sink, DiffLq1, DiffLk1, DiffLq2, DiffLk2, SideEmbed, SideGate, SideProj, SideNorm,
 	Norm1Bias, FinalNormBias, Bigram, VBias, DeltaDecay, DeltaGate,
-	WkvR, WkvMuR, WkvMuK, WkvMuV, WkvMuG, WkvMuW, WkvDecay1, WkvDecay2, WkvDecayBias, WkvBonus, WkvNorm
+	WkvR, WkvMuR, WkvMuK, WkvMuV, WkvMuG, WkvMuW, WkvDecay1, WkvDecay2, WkvDecayBias, WkvBonus, WkvNorm,
+	Talk, WoBias
 };
 
 struct StackSpec {
@@ -233,6 +247,8 @@ struct StackSpec {
 	BigramSpec bigram;
 	int loop_start = 0, loop_stop = 0, loop_times = 1; // layers loop_start .. loop_stop - 1 run loop_times times in a row with the same weights; every
 	                               // pass has its own caches and state, and the embedding output is added to x before every pass but the first
+	int norm_groups = 0;           // > 0: the norms are RMS norms of this many equal neighbouring parts of the vector, each over its own mean square
+	float residual_mult = 1.f;     // x += residual_mult * (sublayer outputs)
 	bool depth_average = false;    // what a layer hands on is a learned weighted sum of the embedding output and all layer results so far
 	// name of a tensor in the checkpoint; `expert` < 0 for tensors that are not per expert
 	std::string (*tensor_name)(int layer, TensorRole role, int expert) = nullptr;

@@ -122,13 +122,19 @@ size_t Config::active_bytes(size_t pos) const {
 				// the packed projection and the output projection(s), the fp32 matrix state read and written, the window of keys
 				total += ((size_t)l.proj_width() + l.mixed_width()) * W * ws + 2 * W * 4;
 				if (l.kind == yalm::MixerKind::StateSpace) total += (size_t)2 * 4 * l.ssm.inner() * l.ssm.state;
+				else if (l.kind == yalm::MixerKind::Retention) total += (size_t)2 * 4 * l.ret.heads * l.ret.dim * l.ret.vdim;
+				else if (l.kind == yalm::MixerKind::LatentAttention) { // second-stage queries, W_uk, W_uv, the window of latents
+					const yalm::LatentSpec &y = l.latent;
+					total += ((size_t)m.heads * (m.dim + y.rot_dim) * y.q_rank + (size_t)m.heads * (m.dim + m.vdim) * y.kv_rank) * ws;
+					total += (m.window > 0 ? std::min<size_t>(pos + 1, m.window) : pos + 1) * (y.kv_rank + y.rot_dim) * cb;
+				} else if (l.kind == yalm::MixerKind::Attention) total += (m.window > 0 ? std::min<size_t>(pos + 1, m.window) : pos + 1) * m.kv_heads * (m.dim + m.vdim) * cb;
 				else {
 					const yalm::DeltaSpec &d = l.delta;
 					total += ((size_t)d.decay_rank * d.heads * d.dim + (size_t)d.gate_rank * d.heads * d.vdim) * ws + (size_t)2 * 4 * d.heads * d.dim * d.vdim;
 					const size_t seen = (m.window > 0 ? std::min<size_t>(pos + 1, m.window) : pos + 1) + (m.window > 0 ? std::min<size_t>(m.keep_first, pos + 1) : 0);
 					total += seen * m.kv_heads * m.dim * cb;
 				}
-				if (l.ffn.kind == yalm::FfnSpec::Moe) total += ((size_t)l.ffn.experts * W + (size_t)l.ffn.top * 3 * l.ffn.ff * W) * ws;
+				if (l.ffn.kind == yalm::FfnSpec::Moe) total += ((size_t)l.ffn.experts * W + (size_t)l.ffn.top * 3 * l.ffn.ff * W + (size_t)3 * l.ffn.shared_ff * W) * ws;
 				continue;
 			}
 			if (s.sandwich_norm) {
@@ -884,7 +890,10 @@ int Model::launches_per_forward(InferenceMode mode) const {
 			} else if (config->stack->sandwich_norm) // norm, projection, mixer (latent 5 with the split merge, differential 4), output projection + norm; norm, up, activation, down + norm; side input
 				n += 2 + (l.kind == yalm::MixerKind::LatentAttention ? 5 : 4) + 1 + (l.ffn.kind == yalm::FfnSpec::None ? 0 : 4) + (config->stack->token_side > 0 ? 1 : 0);
 			else if (config->stack->parallel_block) // norm + shift, projection, mixer (state space 5, parallel 14), experts 3, residual
-				n += 3 + (l.kind == yalm::MixerKind::StateSpace ? 5 : 14) + (l.ffn.kind == yalm::FfnSpec::None ? 0 : 3);
+				n += config->stack->norm_groups > 0 // projection, mixer (latent 7, attention 4, retention 2), experts 3 (+ shared 3), residual + norm
+				         ? 2 + (l.kind == yalm::MixerKind::LatentAttention ? 7 : l.kind == yalm::MixerKind::Attention ? 4 : 2) +
+				               (l.ffn.kind == yalm::FfnSpec::None ? 0 : 3 + (l.ffn.shared_ff > 0 ? 3 : 0))
+				         : 3 + (l.kind == yalm::MixerKind::StateSpace ? 5 : 14) + (l.ffn.kind == yalm::FfnSpec::None ? 0 : 3);
 			else if (l.kind == yalm::MixerKind::LatentAttention || l.kind == yalm::MixerKind::LinearAttention) // norm + conv, projection, mixer (8 / 5), norm + conv, feed-forward (3, or 3 + 3 with a shared expert), depth sum
 				n += 2 + (l.kind == yalm::MixerKind::LatentAttention ? 8 : 5) + 1 +
 				     (l.ffn.kind == yalm::FfnSpec::None ? 0 : 1 + (l.ffn.kind == yalm::FfnSpec::Dense ? 3 : 3 + (l.ffn.shared_ff > 0 ? 3 : 0)));

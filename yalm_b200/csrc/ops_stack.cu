@@ -184,15 +184,15 @@ __global__ void cast_rows_kernel(T *__restrict__ out, const float *__restrict__ 
 // copy in vfirst (the first blending layer), vmode 2 blends v = (1 - lambda) v + lambda vfirst (later blending layers);
 // the blended v is what is cached.  Ring slot of position p: p % ring; caches are head-major (kv head, slot, channel).
 template <typename CT>
-__global__ void __launch_bounds__(256) qkv_post_rows_kernel(float *__restrict__ qkv, int ld, CT *__restrict__ kc, CT *__restrict__ vc,
+__global__ void __launch_bounds__(1024) qkv_post_rows_kernel(float *__restrict__ qkv, int ld, CT *__restrict__ kc, CT *__restrict__ vc,
                                                             float *__restrict__ vfirst, int ldvf, const float *__restrict__ qnorm,
                                                             const float *__restrict__ knorm, const float *__restrict__ vmix, int vmode, int nq,
                                                             int nk, int nv, int dk, int dv, int ring, float eps, int pos0,
-                                                            const int *__restrict__ ctl) {
+                                                            const int *__restrict__ ctl, const float *__restrict__ bias) {
 	__shared__ float red[33];
 	const int m = blockIdx.x, p = first_pos(ctl, pos0) + m;
 	qkv_post_row<CT>(qkv + (size_t)m * ld, kc, vc, vfirst ? vfirst + (size_t)m * ldvf : nullptr, qnorm, knorm, vmix, vmode, nq, nk, nv, dk, dv, ring, p % ring,
-	                 eps, red);
+	                 eps, red, bias);
 }
 
 // Mean key / value (fp32) of every block of `pool` positions whose last position is one of these rows; the members are read
@@ -632,85 +632,88 @@ __global__ void glu_act_rows_kernel(float *__restrict__ h, const float *__restri
 // ---- router ----------------------------------------------------------------------------------------------------------
 // z = Wr x (fp32), scores = sigmoid(z) or softmax(z); the `top` largest (ties: the lower index) with their scores as
 // weights, optionally divided by their sum (+ renorm_eps).  groups > 1: the experts form `groups` equal groups of
-// neighbours, a group scores its best expert, and only experts of the `keep` best groups (ties: the lower index) can be
-// chosen.  One CTA per row; E <= 1024.
+// neighbours, a group is ranked by the sum of its group_top best experts, and only experts of the `keep` best groups (ties: the
+// lower index) can be chosen.  What ranks an expert: its score plus a stored bias, or, without a bias, its logit (both score
+// functions are monotonic, and in fp32 a saturated sigmoid or an underflowed softmax term would tie experts whose exact scores still
+// differ; a sum of two or more experts adds their scores).  Every expert finds its own place: the number of experts before it.  One
+// CTA per row; E <= 1024.
 template <int DT>
 __global__ void __launch_bounds__(256) router_topk_rows_kernel(int *__restrict__ ids, float *__restrict__ wts, const float *__restrict__ x, int ldx,
                                                                const void *__restrict__ wr, int E, int top, int dim, int score, int renorm,
-                                                               float renorm_eps, int groups, int keep, bool vec, const float *__restrict__ bias,
-                                                               float wscale) {
-	extern __shared__ float sc[]; // E, then E logits as they were
+                                                               float renorm_eps, int groups, int keep, int group_top, bool vec,
+                                                               const float *__restrict__ bias, float wscale) {
+	extern __shared__ float sc[]; // E logits, then scores
+	__shared__ float red[33];
+	float *key = sc + E, *gs = key + E, *sel = gs + groups; // E: what ranks an expert; groups; top: the chosen scores
 	const int m = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
 	const float *xr = x + (size_t)m * ldx;
 	for (int e = warp; e < E; e += (int)(blockDim.x >> 5)) {
 		const float z = warp_dot<DT>(wr, (size_t)e * dim, xr, dim, vec);
 		if (lane == 0) sc[e] = z;
 	}
-	float *ch = sc + E + groups; // E: score + bias
 	if (bias)
-		for (int e = threadIdx.x; e < E; e += blockDim.x) ch[e] = bias[e];
+		for (int e = threadIdx.x; e < E; e += blockDim.x) key[e] = bias[e]; // fetched while the products run
 	__syncthreads();
-	if (threadIdx.x == 0) {
-		// The experts are ranked by their logits: both score functions are monotonic, and in fp32 a saturated sigmoid (or an
-		// underflowed softmax term) would tie experts whose exact scores still differ.  Ties go to the lower index.
-		float mx = -INFINITY, sum = 0.f;
-		if (score != 1) {
-			for (int e = 0; e < E; ++e) mx = fmaxf(mx, sc[e]);
-			for (int e = 0; e < E; ++e) sum += expf(sc[e] - mx);
-		}
-		if (groups > 1 && keep < groups) {
-			// a group's rank is its best logit; groups outside the `keep` best lose all their experts
-			float *gbest = sc + E; // groups
-			const int per = E / groups;
-			for (int g = 0; g < groups; ++g) {
+	float mx = 0.f, inv = 1.f;
+	if (score != 1) {
+		float v = -INFINITY, t = 0.f;
+		for (int e = threadIdx.x; e < E; e += blockDim.x) v = fmaxf(v, sc[e]);
+		mx = block_max(v, red);
+		for (int e = threadIdx.x; e < E; e += blockDim.x) t += expf(sc[e] - mx);
+		inv = 1.f / block_sum(t, red);
+	}
+	for (int e = threadIdx.x; e < E; e += blockDim.x) {
+		const float z = sc[e], v = score == 1 ? 1.0f / (1.0f + expf(-z)) : expf(z - mx) * inv;
+		const float k = bias ? v + key[e] : z;
+		sc[e] = v, key[e] = k == k ? k : -INFINITY; // NaN: last, so that the places stay a permutation
+	}
+	__syncthreads();
+	if (groups > 1 && keep < groups) {
+		const int per = E / groups;
+		for (int g = threadIdx.x; g < groups; g += blockDim.x) {
+			float sum = 0.f, above = INFINITY; // the next best below (value, index) of the one before
+			int at = -1;
+			for (int k = 0; k < min(group_top, per); ++k) {
 				float b = -INFINITY;
-				for (int e = g * per; e < (g + 1) * per; ++e) b = fmaxf(b, sc[e]);
-				gbest[g] = b;
+				int bi = per;
+				for (int e = 0; e < per; ++e) {
+					const float v = key[g * per + e];
+					if ((v < above || (v == above && e > at)) && (v > b || bi == per)) b = v, bi = e;
+				}
+				above = b, at = bi;
+				sum += (bias || group_top == 1) ? b : sc[min(g * per + bi, E - 1)];
 			}
-			for (int g = 0; g < groups; ++g) {
-				int better = 0;
-				for (int o = 0; o < groups; ++o) better += (gbest[o] > gbest[g]) || (gbest[o] == gbest[g] && o < g);
-				if (better >= keep)
-					for (int e = g * per; e < (g + 1) * per; ++e) sc[e] = -INFINITY;
-			}
+			gs[g] = sum;
 		}
-		float tot = 0.f;
-		if (bias) {
-			// the choice adds a stored bias to the score, so it cannot be ranked by the logits: rank score + bias, weigh by the score
-			for (int e = 0; e < E; ++e) {
-				sc[e] = sc[e] == -INFINITY ? 0.f : (score == 1 ? 1.0f / (1.0f + expf(-sc[e])) : expf(sc[e] - mx) / sum);
-				ch[e] += sc[e];
-			}
-			for (int j = 0; j < top; ++j) {
-				int best = -1;
-				float bz = -INFINITY;
-				for (int e = 0; e < E; ++e)
-					if (ch[e] > bz) bz = ch[e], best = e;
-				if (best < 0) best = 0;
-				ids[(size_t)m * top + j] = best, wts[(size_t)m * top + j] = sc[best];
-				tot += sc[best];
-				ch[best] = -INFINITY;
-			}
-		} else
-		for (int j = 0; j < top; ++j) {
-			int best = -1;
-			float bz = -INFINITY;
-			for (int e = 0; e < E; ++e)
-				if (sc[e] > bz) bz = sc[e], best = e;
-			if (best < 0) best = 0, bz = sc[0]; // every logit -inf or NaN: keep the indices valid
-			const float bv = score == 1 ? 1.0f / (1.0f + expf(-bz)) : expf(bz - mx) / sum;
-			ids[(size_t)m * top + j] = best, wts[(size_t)m * top + j] = bv;
-			tot += bv;
-			sc[best] = -INFINITY;
+		__syncthreads();
+		for (int e = threadIdx.x; e < E; e += blockDim.x) {
+			const int g = e / per;
+			int better = 0;
+			for (int o = 0; o < groups; ++o) better += (gs[o] > gs[g]) || (gs[o] == gs[g] && o < g);
+			if (better >= keep) key[e] = -INFINITY; // read and written by this thread alone until the next barrier
 		}
-		if (renorm || wscale != 1.f) { // both at once: the weights make one trip to memory and back
-			const float den = renorm ? tot + renorm_eps : 1.f;
-			for (int j = 0; j < top; ++j) {
-				float v = wts[(size_t)m * top + j];
-				if (renorm) v /= den;
-				if (wscale != 1.f) v *= wscale;
-				wts[(size_t)m * top + j] = v;
-			}
+		__syncthreads();
+	}
+	for (int e = threadIdx.x; e < E; e += blockDim.x) {
+		const float k = key[e];
+		int place = 0;
+		for (int o = 0; o < E; ++o) place += (key[o] > k) || (key[o] == k && o < e);
+		if (place < top) ids[(size_t)m * top + place] = e, sel[place] = sc[e];
+	}
+	__syncthreads();
+	if (threadIdx.x < top) { // top <= E; one thread per chosen expert
+		float den = 1.f;
+		if (renorm) {
+			den = renorm_eps;
+			float tot = 0.f;
+			for (int j = 0; j < top; ++j) tot += sel[j];
+			den += tot;
+		}
+		for (int j = threadIdx.x; j < top; j += blockDim.x) {
+			float v = sel[j];
+			if (renorm) v /= den;
+			if (wscale != 1.f) v *= wscale;
+			wts[(size_t)m * top + j] = v;
 		}
 	}
 }
@@ -840,15 +843,24 @@ extern "C" int yalm_cast_rows16(void *out16, const float *x, int ldx, int M, int
 extern "C" int yalm_qkv_post_rows(float *qkv, int ld, void *key_ring, void *value_ring, float *vfirst, int ldvf, const float *qnorm,
                                   const float *knorm, const float *vmix, int vmode, int n, int n_heads, int n_kv, int dk, int dv, int ring,
                                   float eps, int cache_f32, int pos0, const int *ctl, yalm_stream_t s) {
+	return yalm_qkv_bias_post_rows(qkv, ld, nullptr, key_ring, value_ring, vfirst, ldvf, qnorm, knorm, vmix, vmode, n, n_heads, n_kv, dk, dv, ring, eps, cache_f32,
+	                               pos0, ctl, s);
+}
+
+// The same with biases (n_heads dk + n_kv dk + n_kv dv; null: none) added to q, k and v first.
+extern "C" int yalm_qkv_bias_post_rows(float *qkv, int ld, const float *bias, void *key_ring, void *value_ring, float *vfirst, int ldvf, const float *qnorm,
+                                       const float *knorm, const float *vmix, int vmode, int n, int n_heads, int n_kv, int dk, int dv, int ring,
+                                       float eps, int cache_f32, int pos0, const int *ctl, yalm_stream_t s) {
 	if (!qkv || !key_ring || !value_ring || n < 1 || ring < 1 || (vmode && !vfirst) || (vmode == 2 && !vmix)) return YALM_EINVAL;
+	const int threads = n <= 4 ? 1024 : 256; // few rows: one memory round trip per pass over the row
 	const int nq = n_heads * dk, nk = n_kv * dk, nv = n_kv * dv;
 	cudaStream_t st = (cudaStream_t)s;
 	if (cache_f32)
-		qkv_post_rows_kernel<float><<<n, 256, 0, st>>>(qkv, ld, (float *)key_ring, (float *)value_ring, vfirst, ldvf, qnorm, knorm, vmix, vmode, nq, nk,
-		                                               nv, dk, dv, ring, eps, pos0, ctl);
+		qkv_post_rows_kernel<float><<<n, threads, 0, st>>>(qkv, ld, (float *)key_ring, (float *)value_ring, vfirst, ldvf, qnorm, knorm, vmix, vmode, nq, nk,
+		                                               nv, dk, dv, ring, eps, pos0, ctl, bias);
 	else
-		qkv_post_rows_kernel<__nv_bfloat16><<<n, 256, 0, st>>>(qkv, ld, (__nv_bfloat16 *)key_ring, (__nv_bfloat16 *)value_ring, vfirst, ldvf, qnorm,
-		                                                       knorm, vmix, vmode, nq, nk, nv, dk, dv, ring, eps, pos0, ctl);
+		qkv_post_rows_kernel<__nv_bfloat16><<<n, threads, 0, st>>>(qkv, ld, (__nv_bfloat16 *)key_ring, (__nv_bfloat16 *)value_ring, vfirst, ldvf, qnorm,
+		                                                       knorm, vmix, vmode, nq, nk, nv, dk, dv, ring, eps, pos0, ctl, bias);
 	return (int)cudaGetLastError();
 }
 
@@ -1000,7 +1012,7 @@ extern "C" int yalm_glu_act_rows(float *h, const float *gu, int n, int ff, int a
 // score: 0 softmax, 1 sigmoid
 extern "C" int yalm_router_topk_rows(int *ids, float *wts, const float *x, int ldx, const void *wr, int dtype, int n, int n_experts, int top, int dim,
                                      int score, int renorm, float renorm_eps, int groups, int keep_groups, yalm_stream_t s) {
-	return yalm_router_bias_topk_rows(ids, wts, x, ldx, wr, dtype, n, n_experts, top, dim, score, renorm, renorm_eps, groups, keep_groups, nullptr, 1.f, s);
+	return yalm_router_group_topk_rows(ids, wts, x, ldx, wr, dtype, n, n_experts, top, dim, score, renorm, renorm_eps, groups, keep_groups, 1, nullptr, 1.f, s);
 }
 
 // bias (n_experts, optional): the experts are chosen by score + bias, the weights use the score alone; weight_scale multiplies
@@ -1008,12 +1020,19 @@ extern "C" int yalm_router_topk_rows(int *ids, float *wts, const float *x, int l
 extern "C" int yalm_router_bias_topk_rows(int *ids, float *wts, const float *x, int ldx, const void *wr, int dtype, int n, int n_experts, int top, int dim,
                                           int score, int renorm, float renorm_eps, int groups, int keep_groups, const float *bias, float weight_scale,
                                           yalm_stream_t s) {
-	if (!ids || !wts || !x || !wr || n < 1 || top < 1 || top > n_experts || n_experts > 1024 || groups < 1 || n_experts % groups || keep_groups < 1 ||
+	return yalm_router_group_topk_rows(ids, wts, x, ldx, wr, dtype, n, n_experts, top, dim, score, renorm, renorm_eps, groups, keep_groups, 1, bias, weight_scale, s);
+}
+
+// group_top: how many of a group's best experts add up to what ranks the group.
+extern "C" int yalm_router_group_topk_rows(int *ids, float *wts, const float *x, int ldx, const void *wr, int dtype, int n, int n_experts, int top, int dim,
+                                           int score, int renorm, float renorm_eps, int groups, int keep_groups, int group_top, const float *bias,
+                                           float weight_scale, yalm_stream_t s) {
+	if (!ids || !wts || !x || !wr || n < 1 || top < 1 || group_top < 1 || top > n_experts || n_experts > 1024 || groups < 1 || n_experts % groups || keep_groups < 1 ||
 	    keep_groups > groups || top > keep_groups * (n_experts / groups))
 		return YALM_EINVAL;
 	const bool vec = row_vec(wr, dim, dtype) && aligned16(x) && ldx % 4 == 0;
-	DISPATCH_DT(dtype, (router_topk_rows_kernel<DT><<<n, n <= 4 ? 256 : 128, sizeof(float) * (2 * n_experts + groups), (cudaStream_t)s>>>(
-	                       ids, wts, x, ldx, wr, n_experts, top, dim, score, renorm, renorm_eps, groups, keep_groups, vec, bias, weight_scale)));
+	DISPATCH_DT(dtype, (router_topk_rows_kernel<DT><<<n, n <= 4 ? 256 : 128, sizeof(float) * (2 * n_experts + groups + top), (cudaStream_t)s>>>(
+	                       ids, wts, x, ldx, wr, n_experts, top, dim, score, renorm, renorm_eps, groups, keep_groups, group_top, vec, bias, weight_scale)));
 	return (int)cudaGetLastError();
 }
 

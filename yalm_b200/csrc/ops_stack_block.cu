@@ -8,6 +8,7 @@
 //   delta_in_rows       short causal convolutions + SiLU of q, k, v; q, k as unit vectors per head; one decay and one beta per head
 //   wkv_decay_rows      exp(-exp(W_2 tanh(t) + w_0))
 //   block_out_rows      the input of the block's output product: [per-head norm * gate, or the attention's output | act(g) u]
+//   group_norm_rows     x += mult * (sublayer outputs), then an RMS norm over equal parts of the row: one launch between two layers
 //   state_step          a decode row of a matrix-state mixer in one launch, one CTA per head: what feeds the recurrence
 //                       (convolutions and unit norms, or the decay's second stage), one step of it, the head's norm and the gate
 //   gemv_block_in       a decode row's product in: the layer norm (and the blends, by output segment) is applied while the input is staged
@@ -292,8 +293,8 @@ __global__ void __launch_bounds__(256) block_out_rows_kernel(BlockOutArgs a) {
 }
 
 // ---- a decode row of a matrix-state mixer ---------------------------------------------------------------------------------------
-// One CTA per head: (DELTA) convolution + SiLU + unit norms of the head's q and k and of its P channels of v, decay and beta; or
-// (time mixing) the decay's second stage for the head's D channels.  Then one step of the recurrence with the state in the layout
+// One CTA per head: (delta rule) convolution + SiLU + unit norms of the head's q and k and of its P channels of v, decay and beta; or
+// (time mixing) the decay's second stage for the head's D channels; or (retention) the rotation of q and k, with a fixed decay.  Then one step of the recurrence with the state in the layout
 // of state_scan_kernel (8 lanes per column, EPL consecutive rows each), the head's RMS norm, weight and gate.
 struct StateStepArgs {
 	float *out;                   // (H P)
@@ -310,14 +311,18 @@ struct StateStepArgs {
 	const void *w2;               // (H D, rank)
 	const float *w0, *bonus;
 	int rank, vec;
-	const float *norm_w;
+	const float *norm_w;          // null: no weight
 	int w_stride;
 	float eps;
 	int pos0;
 	const int *ctl;
+	const float *decay, *freq;    // retention: (H) decays; rotary frequencies (rot_dims / 2), q_scale is k's factor
+	float rot_mag;
+	int rot_dims, interleaved;
 };
 constexpr int kStepThreads = 512;
-template <int EPL, bool DELTA, int DT>
+constexpr int kStepDelta = 0, kStepBonus = 1, kStepFixed = 2;
+template <int EPL, int MODE, int DT>
 __global__ void __launch_bounds__(kStepThreads) state_step_kernel(StateStepArgs a) {
 	extern __shared__ __align__(16) float sm[];
 	__shared__ float red[33], gates[2];
@@ -350,7 +355,23 @@ __global__ void __launch_bounds__(kStepThreads) state_step_kernel(StateStepArgs 
 	for (int i = tid; i < 4 * DP; i += kStepThreads) sm[i] = 0.f; // rows past D
 	__syncthreads();
 	float decay = 1.f, beta = 0.f;
-	if constexpr (DELTA) {
+	if constexpr (MODE == kStepFixed) {
+		decay = a.decay[h];
+		const int half = a.rot_dims / 2;
+		for (int i = tid; i < D - half; i += kStepThreads) { // a rotated pair, or a channel past the rotated ones
+			const int da = i >= half ? i + half : a.interleaved ? 2 * i : i, db = a.interleaved ? 2 * i + 1 : i + half;
+			float q0 = a.proj[a.o_q + h * D + da], k0 = a.proj[a.o_k + h * D + da];
+			if (i < half) {
+				float q1 = a.proj[a.o_q + h * D + db], k1 = a.proj[a.o_k + h * D + db];
+				rotate_pair(q0, q1, p, a.freq[i], a.rot_mag, &q0, &q1);
+				rotate_pair(k0, k1, p, a.freq[i], a.rot_mag, &k0, &k1);
+				qs[slot(db)] = q1, ks[slot(db)] = k1 * a.q_scale;
+			}
+			qs[slot(da)] = q0, ks[slot(da)] = k0 * a.q_scale;
+		}
+		for (int c = tid; c < P; c += kStepThreads) vs[c] = a.proj[a.o_v + h * P + c];
+		__syncthreads();
+	} else if constexpr (MODE == kStepDelta) {
 		const int g = h / (a.H / a.G), dk = a.G * D, C = 2 * dk + a.H * P;
 		const float *in = a.proj + a.o_q;
 		for (int i = tid; i < 2 * D + P; i += kStepThreads) {
@@ -408,7 +429,13 @@ __global__ void __launch_bounds__(kStepThreads) state_step_kernel(StateStepArgs 
 		if (c0 > 0 && live) load_state(c);
 		const float vv = live ? vs[c] : 0.f;
 		float o4[4] = {0.f, 0.f, 0.f, 0.f};
-		if constexpr (DELTA) {
+		if constexpr (MODE == kStepFixed) {
+#pragma unroll
+			for (int e = 0; e < EPL; ++e) {
+				s[e] = fmaf(decay, s[e], ks[sub * SEG + e] * vv);
+				o4[e & 3] = fmaf(s[e], qs[sub * SEG + e], o4[e & 3]);
+			}
+		} else if constexpr (MODE == kStepDelta) {
 			float d4[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
 			for (int e = 0; e < EPL; ++e) {
@@ -452,7 +479,69 @@ __global__ void __launch_bounds__(kStepThreads) state_step_kernel(StateStepArgs 
 	for (int c = tid; c < P; c += kStepThreads) ss += os[c] * os[c];
 	ss = block_sum(ss, red);
 	const float r = 1.0f / sqrtf(ss / P + a.eps);
-	for (int c = tid; c < P; c += kStepThreads) a.out[h * P + c] = os[c] * r * a.norm_w[h * a.w_stride + c] * act_silu(a.proj[a.o_gate + h * P + c]);
+	for (int c = tid; c < P; c += kStepThreads) a.out[h * P + c] = os[c] * r * (a.norm_w ? a.norm_w[h * a.w_stride + c] : 1.f) * act_silu(a.proj[a.o_gate + h * P + c]);
+}
+
+// ---- residual add + norm in groups ----------------------------------------------------------------------------------------------
+// x += mult * (a + bias + b + sum_j y_j) (whatever is given), then h = x over the root mean square of its group (the row is `groups`
+// equal neighbouring parts), times w; to fp32 rows and / or a 16-bit operand (neither: only the add).  One CTA per row; a warp, or
+// several for few groups, sums a group's squares.  rows: norm only, of x[rows[r]].
+struct GroupNormArgs {
+	float *x;
+	float mult;
+	const float *a, *abias, *b, *y;
+	int ldy, nsum;
+	float *out;
+	void *out16;
+	int bf16;
+	const int *rows;
+	const float *w;
+	int groups, dim;
+	float eps;
+};
+__global__ void __launch_bounds__(1024) group_norm_rows_kernel(GroupNormArgs g) {
+	extern __shared__ __align__(16) float gn_sm[]; // dim values, then partial sums of squares
+	const int m = blockIdx.x, tid = threadIdx.x, nt = blockDim.x, warp = tid >> 5, lane = tid & 31, nw = nt >> 5, dim = g.dim;
+	float *vals = gn_sm, *part = gn_sm + dim;
+	float *xr = g.x + (size_t)(g.rows ? g.rows[m] : m) * dim;
+	const bool add = g.a || g.b || g.y;
+	const size_t o = (size_t)m * dim;
+#pragma unroll 4
+	for (int e = tid; e < dim; e += nt) {
+		float v = xr[e];
+		if (add) {
+			float s = g.a ? g.a[o + e] : 0.f, f = 0.f;
+			if (g.abias) s += g.abias[e];
+			if (g.b) s += g.b[o + e];
+			for (int j = 0; j < g.nsum; ++j) f += g.y[((size_t)m * g.nsum + j) * g.ldy + e];
+			v = fmaf(g.mult, s + f, v);
+			xr[e] = v;
+		}
+		vals[e] = v;
+	}
+	if (!g.w) return;
+	__syncthreads();
+	const int size = dim / g.groups, wpg = max(1, nw / g.groups), slots = nw / wpg; // warps per group, groups in flight
+	if (warp / wpg < slots)
+		for (int k = warp / wpg; k < g.groups; k += slots) {
+			float s = 0.f;
+			for (int e = lane + 32 * (warp % wpg); e < size; e += 32 * wpg) s = fmaf(vals[k * size + e], vals[k * size + e], s);
+			s = warp_sum(s);
+			if (lane == 0) part[k * wpg + warp % wpg] = s;
+		}
+	__syncthreads();
+	for (int k = tid; k < g.groups; k += nt) { // a thread owns its groups' partials
+		float s = 0.f;
+		for (int i = 0; i < wpg; ++i) s += part[k * wpg + i];
+		part[g.groups * wpg + k] = 1.0f / sqrtf(s / size + g.eps);
+	}
+	__syncthreads();
+	const float *r = part + g.groups * wpg;
+	for (int e = tid; e < dim; e += nt) {
+		const float v = vals[e] * r[e / size] * g.w[e];
+		if (g.out) g.out[o + e] = v;
+		if (g.out16) put16(g.out16, o + e, v, g.bf16);
+	}
 }
 
 // ---- a decode row's products ------------------------------------------------------------------------------------------------
@@ -618,6 +707,33 @@ extern "C" int yalm_layer_norm_rows(float *out, void *out16, int bf16, float *x,
 	return (int)cudaGetLastError();
 }
 
+static int launch_group_norm(const GroupNormArgs &g, int n, cudaStream_t st) {
+	if (!g.x || n < 1 || g.dim < 1 || g.groups < 1 || g.dim % g.groups || g.nsum < 0 || (g.nsum && !g.y) || (g.w && !g.out && !g.out16)) return YALM_EINVAL;
+	const int threads = n <= 4 && g.dim > 512 ? 1024 : 256;
+	const size_t smem = sizeof(float) * ((size_t)g.dim + 2 * (size_t)g.groups + threads / 32);
+	if ((int)smem > device_info().max_smem_optin) return YALM_EINVAL;
+	if (smem > 48 * 1024) YALM_TRY(cudaFuncSetAttribute(group_norm_rows_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+	group_norm_rows_kernel<<<n, threads, smem, st>>>(g);
+	return (int)cudaGetLastError();
+}
+
+extern "C" int yalm_group_norm_rows(float *out, void *out16, int bf16, const float *x, const int *rows, const float *w, int groups, float eps, int n, int dim,
+                                    yalm_stream_t s) {
+	if (!w) return YALM_EINVAL;
+	GroupNormArgs g{};
+	g.x = const_cast<float *>(x), g.out = out, g.out16 = out16, g.bf16 = bf16, g.rows = rows, g.w = w, g.groups = groups, g.dim = dim, g.eps = eps;
+	return launch_group_norm(g, n, (cudaStream_t)s);
+}
+
+extern "C" int yalm_residual_group_norm_rows(float *x, float mult, const float *a, const float *a_bias, const float *b, const float *y, int ldy, int nsum,
+                                             float *out, void *out16, int bf16, const float *w, int groups, float eps, int n, int dim, yalm_stream_t s) {
+	if (!a && !b && !y) return YALM_EINVAL;
+	GroupNormArgs g{};
+	g.x = x, g.mult = mult, g.a = a, g.abias = a_bias, g.b = b, g.y = y, g.ldy = ldy, g.nsum = nsum;
+	g.out = out, g.out16 = out16, g.bf16 = bf16, g.w = w, g.groups = groups, g.dim = dim, g.eps = eps;
+	return launch_group_norm(g, n, (cudaStream_t)s);
+}
+
 extern "C" int yalm_mix_rows(float *out, void *out16, int bf16, const float *h, const float *mu, int n_mixes, int plain_mask, float *state, int n, int dim, int pos0,
                              const int *ctl, yalm_stream_t s) {
 	if ((!out && !out16) || !h || !mu || !state || n_mixes < 1 || n_mixes > 31 || n < 1 || dim < 1) return YALM_EINVAL;
@@ -665,16 +781,17 @@ extern "C" int yalm_block_out_rows(float *out, void *out16, int bf16, int ldo, c
 	return (int)cudaGetLastError();
 }
 
-template <bool DELTA>
+template <int MODE>
 static int launch_state_step(const StateStepArgs &a, int dtype, cudaStream_t st) {
 	if (a.D < 1 || a.D > 256 || a.P < 1 || a.H < 1 || a.G < 1 || a.H % a.G) return YALM_EINVAL;
 	const int epl = a.D <= 8 ? 1 : a.D <= 16 ? 2 : a.D <= 32 ? 4 : a.D <= 64 ? 8 : a.D <= 128 ? 16 : 32;
-	const size_t smem = sizeof(float) * (4 * (size_t)8 * (epl + (epl >= 8 ? 4 : 0)) + a.P + std::max(a.P, DELTA ? 0 : a.rank));
+	const size_t smem = sizeof(float) * (4 * (size_t)8 * (epl + (epl >= 8 ? 4 : 0)) + a.P + std::max(a.P, MODE == kStepBonus ? a.rank : 0));
 	if (smem > 48 * 1024) return YALM_EINVAL;
-#define STEP_DT(EPL_, DT_) state_step_kernel<EPL_, DELTA, DT_><<<a.H, kStepThreads, smem, st>>>(a)
+#define STEP_DT(EPL_, DT_) state_step_kernel<EPL_, MODE, DT_><<<a.H, kStepThreads, smem, st>>>(a)
 #define STEP_CASE(EPL_)                                             \
 	{                                                               \
-		if (DELTA || dtype == YALM_F32) STEP_DT(EPL_, YALM_F32);    \
+		if constexpr (MODE != kStepBonus) STEP_DT(EPL_, YALM_F32);  \
+		else if (dtype == YALM_F32) STEP_DT(EPL_, YALM_F32);        \
 		else if (dtype == YALM_F16) STEP_DT(EPL_, YALM_F16);        \
 		else if (dtype == YALM_BF16) STEP_DT(EPL_, YALM_BF16);      \
 		else return YALM_EINVAL;                                    \
@@ -698,7 +815,7 @@ extern "C" int yalm_delta_step(float *out, float *state, const float *proj, int 
 	a.out = out, a.state = state, a.proj = proj, a.o_q = o_qkv, a.o_gate = o_gate, a.o_beta = o_beta, a.o_decay = o_decay;
 	a.H = heads, a.G = kv_heads, a.D = dim, a.P = vdim, a.conv_w = conv_w, a.ring = ring, a.taps = taps, a.a_log = a_log, a.dt_bias = dt_bias;
 	a.unit_eps = unit_eps, a.q_scale = q_scale, a.norm_w = norm_w, a.w_stride = 0, a.eps = eps, a.pos0 = pos0, a.ctl = ctl;
-	return launch_state_step<true>(a, YALM_F32, (cudaStream_t)s);
+	return launch_state_step<kStepDelta>(a, YALM_F32, (cudaStream_t)s);
 }
 
 extern "C" int yalm_wkv_step(float *out, float *state, const float *proj, int o_r, int o_k, int o_v, int o_gate, int o_decay, const void *w2, const float *w0,
@@ -710,7 +827,18 @@ extern "C" int yalm_wkv_step(float *out, float *state, const float *proj, int o_
 	a.H = heads, a.G = heads, a.D = dim, a.P = dim, a.w2 = w2, a.w0 = w0, a.bonus = bonus, a.rank = rank;
 	a.vec = al16(w2) && rank % (dtype == YALM_F32 ? 4 : 8) == 0;
 	a.norm_w = norm_w, a.w_stride = dim, a.eps = eps, a.pos0 = pos0, a.ctl = ctl;
-	return launch_state_step<false>(a, dtype, (cudaStream_t)s);
+	return launch_state_step<kStepBonus>(a, dtype, (cudaStream_t)s);
+}
+
+extern "C" int yalm_retention_step(float *out, float *state, const float *proj, int o_q, int o_k, int o_v, int o_gate, const float *decay, const float *freq,
+                                   float magnitude, int rot_dims, int interleaved, float k_scale, int heads, int dim, int vdim, float eps, int pos0, const int *ctl,
+                                   yalm_stream_t s) {
+	if (!out || !state || !proj || !decay || rot_dims < 0 || rot_dims % 2 || rot_dims > dim || (rot_dims > 0 && !freq)) return YALM_EINVAL;
+	StateStepArgs a{};
+	a.out = out, a.state = state, a.proj = proj, a.o_q = o_q, a.o_k = o_k, a.o_v = o_v, a.o_gate = o_gate;
+	a.H = heads, a.G = heads, a.D = dim, a.P = vdim, a.q_scale = k_scale, a.eps = eps, a.pos0 = pos0, a.ctl = ctl;
+	a.decay = decay, a.freq = freq, a.rot_mag = magnitude, a.rot_dims = rot_dims, a.interleaved = interleaved;
+	return launch_state_step<kStepFixed>(a, YALM_F32, (cudaStream_t)s);
 }
 
 extern "C" int yalm_gemv_block_in(float *out, const float *x, const void *w, int n, int d, int dtype, const float *norm_w, const float *norm_b, float eps,

@@ -149,17 +149,6 @@ __global__ void norm_conv_state_kernel(float *state, const float *__restrict__ h
 	}
 }
 
-// ---- rotary positions ---------------------------------------------------------------------------------------------------
-// Pair i of a vector at position p turns by p * freq[i]; cos and sin carry the magnitude factor.  Position, angle and the
-// rotation are fp32.  interleaved: the pair is (2 i, 2 i + 1), else (i, i + half).
-__device__ __forceinline__ void rotate_pair(float a, float b, int p, float freq, float mag, float *ra, float *rb) {
-	const float ang = (float)p * freq;
-	float sn, cs;
-	sincosf(ang, &sn, &cs);
-	sn *= mag, cs *= mag;
-	*ra = a * cs - b * sn, *rb = b * cs + a * sn;
-}
-
 // ---- latent attention: norms, rotation, cache append ----------------------------------------------------------------------
 // Row m of the packed projection P (ld): [o_q, +q_rank) the query latent: RMS norm with weight qw in place.  With a cache of
 // its own, [o_kv, +kv_rank) RMS-normed with weight kw is the key / value latent and [o_kv + kv_rank, +rot_dim) the shared key
@@ -539,9 +528,9 @@ __global__ void __launch_bounds__(kLaWarps * 32) attn_latent_rows_kernel(float *
 	}
 }
 // out[m, h, :] = sum_z w_z acc_z / sum_z w_z L_z with w_z = exp(M_z - max M), splits taken in order (a split without keys has
-// M = -inf and no weight).  grid (heads, rows).
+// M = -inf and no weight); with a gate (one number per row and head) times sigmoid(gate).  grid (heads, rows).
 __global__ void attn_latent_merge_kernel(float *__restrict__ out, int ldo, const float *__restrict__ part, int n_heads, int dv, int nsplit,
-                                         const float *__restrict__ sink) {
+                                         const float *__restrict__ sink, const float *__restrict__ gate = nullptr, int ldg = 0) {
 	__shared__ float wz[128]; // the splits' weights over the common sum (nsplit <= 128)
 	const int h = blockIdx.x, m = blockIdx.y;
 	const float *pr = part + (size_t)(m * n_heads + h) * nsplit * (dv + 2);
@@ -561,7 +550,8 @@ __global__ void attn_latent_merge_kernel(float *__restrict__ out, int ldo, const
 		// the sum runs over the splits in order
 		float L = 0.f;
 		for (int z = 0; z < nsplit; ++z) L += __shfl_sync(kFull, z < 32 ? t[0] : z < 64 ? t[1] : z < 96 ? t[2] : t[3], z & 31);
-		const float fin = softmax_finish(M, L, sink, h);
+		float fin = softmax_finish(M, L, sink, h);
+		if (gate) fin /= 1.0f + expf(-gate[(size_t)m * ldg + h]);
 #pragma unroll
 		for (int k = 0; k < 4; ++k)
 			if (lane + 32 * k < nsplit) wz[lane + 32 * k] = e[k] * fin;
@@ -780,9 +770,14 @@ extern "C" int yalm_attn_latent_rows_sink(float *out, int ldo, const float *q, i
 	return YALM_EINVAL;
 }
 
-// Joins nsplit (<= 128) partials per (row, head) of (dv accumulators, max, sum) in `part`, in order, sink included (null: none).
-extern "C" int yalm_attn_latent_merge(float *out, int ldo, const float *part, int n, int n_heads, int dv, int nsplit, const float *sink, yalm_stream_t s) {
+// Joins nsplit (<= 128) partials per (row, head) of (dv accumulators, max, sum) in `part`, in order, sink included (null: none);
+// gate (n, n_heads; row stride ldg; null: none): every head's result times sigmoid(gate).
+extern "C" int yalm_attn_split_merge(float *out, int ldo, const float *part, int n, int n_heads, int dv, int nsplit, const float *sink, const float *gate,
+                                     int ldg, yalm_stream_t s) {
 	if (!out || !part || n < 1 || n_heads < 1 || dv < 1 || nsplit < 1 || nsplit > 128) return YALM_EINVAL;
-	attn_latent_merge_kernel<<<dim3(n_heads, n, (dv + 127) / 128), 128, 0, (cudaStream_t)s>>>(out, ldo, part, n_heads, dv, nsplit, sink);
+	attn_latent_merge_kernel<<<dim3(n_heads, n, (dv + 127) / 128), 128, 0, (cudaStream_t)s>>>(out, ldo, part, n_heads, dv, nsplit, sink, gate, ldg);
 	return (int)cudaGetLastError();
+}
+extern "C" int yalm_attn_latent_merge(float *out, int ldo, const float *part, int n, int n_heads, int dv, int nsplit, const float *sink, yalm_stream_t s) {
+	return yalm_attn_split_merge(out, ldo, part, n, n_heads, dv, nsplit, sink, nullptr, 0, s);
 }

@@ -393,7 +393,7 @@ __global__ void __launch_bounds__(128) head_norm_gate_rows_kernel(float *__restr
 	const float r = 1.0f / sqrtf(ss / P + eps);
 	for (int c = lane; c < P; c += 32) {
 		const float g = gate[(size_t)m * ldg + h * P + c];
-		out[(size_t)m * ldo + h * P + c] = row[c] * r * w[c] * (gate_silu ? siluf_(g) : sigmoidf_(g));
+		out[(size_t)m * ldo + h * P + c] = row[c] * r * (w ? w[c] : 1.f) * (gate_silu ? siluf_(g) : sigmoidf_(g));
 	}
 }
 
@@ -773,10 +773,10 @@ extern "C" int yalm_head_norm_gate_rows(float *out, int ldo, const float *o, int
 	return yalm_head_norm_act_rows(out, ldo, o, ldi, gate, ldg, w, n, heads, vdim, eps, 0, s);
 }
 
-// gate_silu != 0: the gate is silu(gate) instead of sigmoid(gate)
+// gate_silu != 0: the gate is silu(gate) instead of sigmoid(gate); w null: no weight
 extern "C" int yalm_head_norm_act_rows(float *out, int ldo, const float *o, int ldi, const float *gate, int ldg, const float *w, int n, int heads, int vdim,
                                        float eps, int gate_silu, yalm_stream_t s) {
-	if (!out || !o || !gate || !w || n < 1 || heads < 1 || vdim < 1) return YALM_EINVAL;
+	if (!out || !o || !gate || n < 1 || heads < 1 || vdim < 1) return YALM_EINVAL;
 	head_norm_gate_rows_kernel<<<dim3((heads + 3) / 4, n), 128, 0, (cudaStream_t)s>>>(out, ldo, o, ldi, gate, ldg, w, heads, vdim, eps, gate_silu);
 	return (int)cudaGetLastError();
 }

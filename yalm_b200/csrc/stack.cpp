@@ -106,6 +106,10 @@ struct StackLayer {
 	std::vector<int> seg_end;                                 // output columns of every segment of wproj
 	int plain_mask = 0;                                       // segments that read the norm's output itself
 	bool add_embedding = false;                               // the embedding output is added to x right before this layer run
+	// ---- parallel blocks: retention (columns [q | k | v | gate]), attention with mixed head scores (columns [q | k | v | one gate per head]) ----
+	float *decay = nullptr, *k_scale = nullptr;               // (heads) each
+	float *talk = nullptr, *o_bias = nullptr;                 // (heads, heads), (dim)
+	int n_bias = 0;                                           // entries per head of bias_table where it stops at rel_far
 	const StackLayer *shares = nullptr;                       // a repeated pass of that layer: its weights, own caches and state
 	void *side_gate = nullptr, *side_proj = nullptr;          // token side input: (token_side, dim), (dim, token_side)
 	float *side_norm = nullptr;
@@ -226,6 +230,13 @@ uint16_t narrow_bf16(float f) { // round to nearest even
 
 } // namespace
 
+// Row of a table of `rows` distance biases for distance n: exact below rows / 2, logarithmic up to `far`, then the last row.
+static int distance_bucket(int n, int rows, int far) {
+	const int half = rows / 2;
+	if (n < half) return n;
+	return std::min(rows - 1, half + (int)std::floor(std::log((double)n / half) / std::log((double)far / half) * (rows - half)));
+}
+
 // Host bytes of tensor `t` in dtype `want` (the tensor's own bytes when it already is; else converted into a buffer the
 // model keeps until the upload).  Supported: anything -> F32, F32 -> BF16.
 static const void *host_as(std::vector<std::vector<char>> &keep, const Tensor *t, DType want, size_t numel) {
@@ -272,6 +283,9 @@ struct Model::StackScratch {
 	void *lat16 = nullptr, *lat_ek = nullptr, *lat_ev = nullptr; // latent attention, prompt portions: latents of the visible rows (bf16), keys / values per head
 	float *latkv = nullptr;
 	float *attn_ws = nullptr; // split partials of decode-sized attention calls
+	float *mixed_ws = nullptr; // split partials of the attention with mixed head scores
+	size_t mixed_floats = 0;
+	void *n16 = nullptr;      // norms in groups, prompt portions: the normed rows as the 16-bit operand of several products
 	int *ids = nullptr, *tokens = nullptr, *want = nullptr, *targets = nullptr;
 	float *moe_gu = nullptr, *moe_ys = nullptr; // experts on the tensor cores: (gate | up) and down outputs of the slots sorted by expert
 	int *order = nullptr;                       // slot at every place of that order
@@ -486,6 +500,14 @@ void Model::build_stack(YALMData &data) {
 			_stack.push_back(L);
 			continue;
 		}
+		auto rotary_table = [&](const yalm::RotarySpec &rot) {
+			if (rot.dims < 1) return;
+			std::vector<float> fr;
+			rot.table(&fr, &L->rot_mag);
+			_host_converted.emplace_back(fr.size() * sizeof(float));
+			memcpy(_host_converted.back().data(), fr.data(), fr.size() * sizeof(float));
+			pl.push_back({(void **)&L->rot_freq, {{_host_converted.back().data(), fr.size() * sizeof(float)}}});
+		};
 		if (s.parallel_block) {
 			// ---- one norm, a packed projection of the mixer's input, per-mixer pieces, experts ----
 			const int W = s.width;
@@ -530,13 +552,11 @@ void Model::build_stack(YALMData &data) {
 				pl.push_back({(void **)&L->head_bias, {vec32(tensor(i, TensorRole::HeadBias, -1, {m.heads}))}});
 				pl.push_back({&L->wo, {mat(tensor(i, TensorRole::Wo, -1, {W, no}))}});
 				{ // distance -> table row: exact below rows / 2, logarithmic up to rel_far, then the last row
-					const int rows = m.rel_rows, half = rows / 2;
-					if (m.rel_far <= half) die("distance bias: the farthest bucketed distance must exceed half the table");
+					const int rows = m.rel_rows;
+					if (m.rel_far <= rows / 2) die("distance bias: the farthest bucketed distance must exceed half the table");
 					_host_converted.emplace_back((size_t)c.max_seq_len * sizeof(int));
 					int *b = reinterpret_cast<int *>(_host_converted.back().data());
-					for (int n = 0; n < c.max_seq_len; ++n)
-						b[n] = n < half ? n
-						                : std::min(rows - 1, half + (int)std::floor(std::log((double)n / half) / std::log((double)m.rel_far / half) * (rows - half)));
+					for (int n = 0; n < c.max_seq_len; ++n) b[n] = distance_bucket(n, rows, m.rel_far);
 					pl.push_back({(void **)&L->bucket, {{b, (size_t)c.max_seq_len * sizeof(int)}}});
 					const float *rel32 = static_cast<const float *>(vec32(tensor(i, TensorRole::RelBias, -1, {m.rel_rows, m.heads})).first);
 					const float *hb32 = static_cast<const float *>(vec32(tensor(i, TensorRole::HeadBias, -1, {m.heads})).first);
@@ -562,8 +582,57 @@ void Model::build_stack(YALMData &data) {
 				const size_t cb = c.weight_dtype == DType::F32 ? 4 : 2;
 				L->state_allocs.push_back({&L->kring, (size_t)m.kv_heads * L->ring * m.dim * cb});
 				if (m.window > 0 && m.keep_first > 0) L->state_allocs.push_back({&L->kfirst, (size_t)m.kv_heads * m.keep_first * m.dim * cb});
+			} else if (ls.kind == yalm::MixerKind::LatentAttention) {
+				load_latent(i, L, proj, W);
+			} else if (ls.kind == yalm::MixerKind::Retention) {
+				const yalm::RetentionSpec &r = ls.ret;
+				const int hd = r.heads * r.dim, hp = r.heads * r.vdim;
+				if (r.dim > 256) die("retention: key sizes above 256 are not built");
+				L->o_q = 0, L->o_k = hd, L->o_v = 2 * hd, L->o_gate = 2 * hd + hp;
+				proj.parts.push_back(mat(tensor(i, TensorRole::Wq, -1, {hd, W})));
+				proj.parts.push_back(mat(tensor(i, TensorRole::Wk, -1, {hd, W})));
+				proj.parts.push_back(mat(tensor(i, TensorRole::Wv, -1, {hp, W})));
+				proj.parts.push_back(mat(tensor(i, TensorRole::OutGate, -1, {hp, W})));
+				pl.push_back({&L->wo, {mat(tensor(i, TensorRole::Wo, -1, {W, hp}))}});
+				_host_converted.emplace_back((size_t)2 * r.heads * sizeof(float));
+				float *c2 = reinterpret_cast<float *>(_host_converted.back().data());
+				for (int hh = 0; hh < r.heads; ++hh) c2[hh] = r.decay[hh], c2[r.heads + hh] = 1.0f / sqrtf((float)r.dim);
+				pl.push_back({(void **)&L->decay, {{c2, (size_t)r.heads * sizeof(float)}}});
+				pl.push_back({(void **)&L->k_scale, {{c2 + r.heads, (size_t)r.heads * sizeof(float)}}});
+				rotary_table(r.rot);
+				L->state_allocs.push_back({(void **)&L->scan_state, (size_t)r.heads * r.vdim * r.dim * 4});
+			} else if (ls.kind == yalm::MixerKind::Attention && m.talk) {
+				const int nq = m.heads * m.dim, nk = m.kv_heads * m.dim, nv = m.kv_heads * m.vdim, no = m.heads * m.vdim;
+				L->o_q = 0, L->o_k = nq, L->o_v = nq + nk, L->o_gate = nq + nk + nv;
+				proj.parts.push_back(mat(tensor(i, TensorRole::Wq, -1, {nq, W})));
+				proj.parts.push_back(mat(tensor(i, TensorRole::Wk, -1, {nk, W})));
+				proj.parts.push_back(mat(tensor(i, TensorRole::Wv, -1, {nv, W})));
+				if (m.head_gate) proj.parts.push_back(mat(tensor(i, TensorRole::OutGate, -1, {m.heads, W})));
+				if (m.qk_bias && m.v_bias)
+					pl.push_back({(void **)&L->qkb, {vec32(tensor(i, TensorRole::QBias, -1, {nq})), vec32(tensor(i, TensorRole::KBias, -1, {nk})), vec32(tensor(i, TensorRole::VBias, -1, {nv}))}});
+				if (m.qk_norm == yalm::QkNorm::WholeProjection) {
+					pl.push_back({(void **)&L->qnorm, {vec32(tensor(i, TensorRole::QNorm, -1, {nq}))}});
+					pl.push_back({(void **)&L->knorm, {vec32(tensor(i, TensorRole::KNorm, -1, {nk}))}});
+				}
+				if (m.o_bias) pl.push_back({(void **)&L->o_bias, {vec32(tensor(i, TensorRole::WoBias, -1, {W}))}});
+				pl.push_back({(void **)&L->talk, {vec32(tensor(i, TensorRole::Talk, -1, {m.heads, m.heads}))}});
+				pl.push_back({&L->wo, {mat(tensor(i, TensorRole::Wo, -1, {W, no}))}});
+				if (m.rel_rows > 0) { // per head, the bias of every distance up to rel_far, from where on it is the last row's
+					if (m.rel_far <= m.rel_rows / 2) die("distance bias: the farthest bucketed distance must exceed half the table");
+					const float *rel32 = static_cast<const float *>(vec32(tensor(i, TensorRole::RelBias, -1, {m.rel_rows, m.heads})).first);
+					L->n_bias = m.rel_far + 1;
+					_host_converted.emplace_back((size_t)m.heads * L->n_bias * sizeof(float));
+					float *tb = reinterpret_cast<float *>(_host_converted.back().data());
+					for (int hh = 0; hh < m.heads; ++hh)
+						for (int n = 0; n < L->n_bias; ++n) tb[(size_t)hh * L->n_bias + n] = rel32[(size_t)distance_bucket(n, m.rel_rows, m.rel_far) * m.heads + hh];
+					pl.push_back({(void **)&L->bias_table, {{tb, (size_t)m.heads * L->n_bias * sizeof(float)}}});
+				}
+				L->ring = m.window > 0 ? std::min(c.max_seq_len, (m.window + c.stack_chunk + 63) / 64 * 64) : c.max_seq_len;
+				const size_t cb = c.weight_dtype == DType::F32 ? 4 : 2;
+				L->state_allocs.push_back({&L->kring, (size_t)m.kv_heads * L->ring * m.dim * cb});
+				L->state_allocs.push_back({&L->vring, (size_t)m.kv_heads * L->ring * m.vdim * cb});
 			} else
-				die("parallel blocks take a state-space or a parallel mixer");
+				die("parallel blocks take a state-space mixer, a parallel one, latent attention, retention, or attention with mixed head scores");
 			pl.push_back(proj);
 			const FfnSpec &f = ls.ffn;
 			if (f.kind == FfnSpec::Moe) {
@@ -575,6 +644,12 @@ void Model::build_stack(YALMData &data) {
 				}
 				pl.push_back(g), pl.push_back(u), pl.push_back(dn);
 				pl.push_back({&L->router, {mat(tensor(i, TensorRole::Router, -1, {f.experts, W}))}});
+				if (f.choice_bias) pl.push_back({(void **)&L->router_bias, {vec32(tensor(i, TensorRole::RouterBias, -1, {f.experts}))}});
+				if (f.shared_ff > 0) {
+					if (ls.kind == yalm::MixerKind::Parallel) die("a shared expert beside two mixers is not built");
+					pl.push_back({&L->wsgu, {mat(tensor(i, TensorRole::SharedGate, -1, {f.shared_ff, W})), mat(tensor(i, TensorRole::SharedUp, -1, {f.shared_ff, W}))}});
+					pl.push_back({&L->wsdown, {mat(tensor(i, TensorRole::SharedDown, -1, {W, f.shared_ff}))}});
+				}
 			} else if (f.kind != FfnSpec::None)
 				die("parallel blocks take experts or no feed-forward");
 			_stack.push_back(L);
@@ -870,7 +945,7 @@ void Model::cuda_stack(int device) {
 		const yalm::LayerSpec &ls = L->spec;
 		if (ls.kind != yalm::MixerKind::LatentAttention) continue;
 		if (ls.mix.dim > 0 && !L->wuv) L->wuv = static_cast<char *>(L->wuk) + (size_t)ls.mix.heads * ls.mix.dim * ls.latent.kv_rank * dtype_size(c.weight_dtype);
-		if (c.weight_dtype == DType::F32 || (ls.mix.window < 1 && !L->sandwich)) continue;
+		if (c.weight_dtype == DType::F32) continue;
 		// the rows a portion sees: the window before it and itself, or (no window) everything the ring holds
 		const size_t rows = ls.mix.window > 0 ? std::min<size_t>(L->ring, (size_t)ls.mix.window + c.stack_chunk) : (size_t)L->ring, H = ls.mix.heads;
 		lat16 = std::max(lat16, rows * ls.latent.kv_rank * 2), latkv = std::max(latkv, rows * H * (ls.mix.dim + ls.mix.vdim) * 4);
@@ -884,6 +959,8 @@ void Model::cuda_stack(int device) {
 	int mixes = 1;
 	for (auto &L : _stack)
 		if (L->spec.kind == yalm::MixerKind::TimeMix) time_mix = true, mixes = std::max(mixes, (int)L->seg_end.size());
+	for (auto &L : _stack)
+		if (L->talk) S.mixed_floats = std::max(S.mixed_floats, yalm_attn_mixed_workspace(c.stack_chunk, L->spec.mix.heads, L->spec.mix.vdim));
 	const size_t blk = s.packed_block ? s.max_block_out() : 0;
 	const bool moe = s.max_experts() > 0 && c.weight_dtype != DType::F32; // the grouped route needs 16-bit operands
 	auto pad = [](size_t b) { return (b + 255) / 256 * 256; };
@@ -897,6 +974,7 @@ void Model::cuda_stack(int device) {
 	             {(void **)&S.a16, 2 * cap * std::max({top * kmax, blk, mixes * W})}, {(void **)&S.a16e, pb * 2 * cap * top * kmax}, {(void **)&S.a16r, pb * 2 * cap * top * kmax}, {(void **)&S.ids, 4 * cap * top},       {(void **)&S.tokens, 4 * cap},
 	             {(void **)&S.want, 4 * cap},            {(void **)&S.targets, 4 * cap},
 	             {(void **)&S.attn_ws, 4 * yalm_attn_window_pool_workspace(512)}, {(void **)&S.ticket, 256},
+	             {(void **)&S.mixed_ws, 4 * S.mixed_floats}, {(void **)&S.n16, s.norm_groups > 0 ? 2 * cap * W : 0},
 	             {(void **)&S.hs, pb * 4 * cap * W}, {(void **)&S.conv, pb * 4 * cap * nconv}, {(void **)&S.aux, pb * 4 * cap * naux},
 	             {(void **)&S.scan, pb * 4 * cap * no}, {(void **)&S.att2, pb * 4 * cap * no}, {(void **)&S.y1, pb * 4 * cap * W}, {(void **)&S.y2, pb * 4 * cap * W},
 	             {(void **)&S.hist, 4 * cap * W * (size_t)S.hist_slabs}, {(void **)&S.hsh, 4 * cap * shared_ff},
@@ -1019,20 +1097,91 @@ int Model::stack_moe_grouped(StackScratch &S, const yalm::StackLayer &L, const f
 	return (int)cudaGetLastError(); // `order` was pageable host memory: the copy call returned after staging it
 }
 
-// One parallel block over n rows: h = norm(x); the mixer reads the token-shifted h through ONE packed projection, the experts
-// read h itself; x += mixer + experts.  What the rows leave for the next call (previous h, convolution tails, matrix states,
+static int glu_act_code(yalm::GluAct a) {
+	return a == yalm::GluAct::SigmoidScaled ? 2 : a == yalm::GluAct::GeluTanh ? 3 : a == yalm::GluAct::Silu ? YALM_ACT_SILU : YALM_ACT_GELU;
+}
+
+// The same product when the rows already exist as a 16-bit operand (h16 null, or sizes the tensor-core product does not take: from x).
+static int stack_linear_h(Model &m, const Config &c, void *a16, const void *h16, float *y, int ldy, const float *x, int ldx, const void *w, int M, int N, int K,
+                          cudaStream_t st) {
+	if (h16 && ldy % 4 == 0 && ((uintptr_t)y & 15) == 0 && ((uintptr_t)w & 15) == 0) return yalm_gemm_16(y, ldy, h16, w, M, N, K, 0, c.weight_dtype == DType::BF16, 1.f, st);
+	return stack_linear(m, c, a16, y, ldy, x, ldx, w, M, N, K, 1.f, st);
+}
+
+// Latent attention over n rows of the packed projection P (columns as load_latent laid them out), up to the output projection: the
+// heads' outputs go to S.att.  The cache rows are [latent | rotated key part], the layer's own or another layer's.
+int Model::stack_latent(StackScratch &S, const yalm::StackLayer &L, float *P, int ldp, int n, int pos0, const int *ctl, cudaStream_t st) {
+	const Config &c = *config;
+	const yalm::LayerSpec &ls = L.spec;
+	const yalm::MixerSpec &m = ls.mix;
+	const yalm::LatentSpec &a = ls.latent;
+	const float eps = c.stack->norm_eps;
+	const int dt = static_cast<int>(c.weight_dtype), f32 = c.weight_dtype == DType::F32, inter = a.rot.interleaved ? 1 : 0;
+	const int row = a.kv_rank + a.rot_dim, nq = m.heads * (m.dim + a.rot_dim), nqa = m.heads * row, nl = m.heads * a.kv_rank, no = m.heads * m.vdim, dk = m.dim + a.rot_dim;
+	const bool own = a.kv_from < 0;
+	if (own || a.q_rank > 0)
+		ST_TRY(yalm_latent_post_rows(P, ldp, L.o_q, a.q_rank, L.qnorm, L.o_kv, a.kv_rank, a.rot_dim, L.knorm, own ? L.kring : nullptr, L.ring, L.rot_freq, L.rot_mag,
+		                             a.rot.dims, inter, eps, f32, n, pos0, ctl, st));
+	float *Q = P + L.o_q; // the queries as projected, per head [unrotated | rotated part]
+	int ldq = ldp;
+	if (a.q_rank > 0) {
+		ST_TRY(stack_linear(*this, c, S.a16, S.conv, nq, Q, ldp, L.wuq, n, nq, a.q_rank, 1.f, st));
+		Q = S.conv, ldq = nq;
+	}
+	if (!f32 && !ctl && n >= 16 && m.dim > 0 && S.lat16 && a.kv_rank % 8 == 0 && ldq % 4 == 0 && L.o_q % 4 == 0 && no % 2 == 0 && (m.heads * (m.dim + m.vdim)) % 4 == 0 &&
+	    yalm_attn_window_pool_mma_shape(dk, m.vdim) && !attn_mma_off()) {
+		// A prompt portion in 16-bit: the latents of the visible rows times [W_uk ; W_uv] on the tensor cores give every head's keys
+		// and values, written beside the rotated key part into head-major rings for the tensor-core attention; the queries stay as
+		// projected, their rotated part turned in place.
+		const int first = m.window > 0 ? std::max(0, pos0 - m.window + 1) : 0, count = pos0 + n - first, nkv = m.heads * (m.dim + m.vdim);
+		ST_TRY(yalm_latent_gather_rows16(S.lat16, L.kring, L.ring, row, a.kv_rank, first, count, st));
+		ST_TRY(yalm_gemm_16(S.latkv, nkv, S.lat16, L.wuk, count, nkv, a.kv_rank, 0, dt == YALM_BF16, 1.f, st));
+		ST_TRY(yalm_latent_pack_rings(S.lat_ek, S.lat_ev, S.latkv, nkv, L.kring, L.ring, a.kv_rank, a.rot_dim, m.heads, m.dim, m.vdim, L.ring, first, count, st));
+		ST_TRY(yalm_rotate_heads_rows(Q, ldq, m.heads, dk, m.dim, L.rot_freq, L.rot_mag, a.rot.dims, inter, n, pos0, ctl, st));
+		ST_TRY(yalm_attn_window_pool_mma_sink(S.att, no, Q, ldq, S.lat_ek, S.lat_ev, nullptr, nullptr, n, m.heads, m.heads, dk, m.vdim, L.ring, 0, m.window, 0, m.scale,
+		                                      pos0, ctl, L.sink, m.heads, st));
+		if (m.out_gate) ST_TRY(yalm_sigmoid_gate_rows(S.att, no, P + L.o_gate, ldp, n, no, st));
+		return 0;
+	}
+	// A decode row (and what the tensor-core route does not take): W_uk moves to the query side, every head reads the one cached row of a
+	// position — keys are whole rows, values their first kv_rank channels — and W_uv follows the weighted sum.
+	ST_TRY(yalm_latent_query_rows(S.aux, nqa, Q, ldq, L.wukt, dt, n, m.heads, m.dim, a.rot_dim, a.kv_rank, L.rot_freq, L.rot_mag, a.rot.dims, inter, pos0, ctl, st));
+	static const bool latent_mma_off = [] { const char *e = getenv("YALM_STACK_LATENT_MMA"); return e && e[0] == '0'; }(); // A/B against the SIMT kernels
+	static const bool one_pass_off = [] { const char *e = getenv("YALM_STACK_ATTN_LANES"); return e && e[0] == '0'; }();
+	const bool rows16 = !f32 && ((uintptr_t)L.kring & 15) == 0 && nqa % 4 == 0;
+	if (rows16 && !latent_mma_off && yalm_attn_latent_mma_shape(row, a.kv_rank, row) && n * m.heads <= 4096) {
+		// the heads as the M tile of the tensor cores; the keys a row can ever see, in tiles of 64, are split over up to 128 CTAs (shapes only)
+		const int tiles = ((m.window > 0 ? std::min(m.window, c.max_seq_len) : c.max_seq_len) + 63) / 64, ctas = (m.heads + 15) / 16 * n;
+		const int cap = std::max(1, std::min({tiles, 128, 4096 / (n * m.heads), (296 + ctas - 1) / ctas}));
+		const int per = (tiles + cap - 1) / cap, nsplit = (tiles + per - 1) / per;
+		ST_TRY(yalm_attn_latent_mma_rows(S.scan, nl, S.aux, nqa, L.kring, row, S.attn_ws, n, m.heads, row, a.kv_rank, L.ring, m.window, m.scale, nsplit, pos0, ctl, L.sink,
+		                                 st));
+	} else if (rows16 && !one_pass_off && yalm_attn_latent_rows_shape(row, a.kv_rank, row))
+		ST_TRY(yalm_attn_latent_rows_sink(S.scan, nl, S.aux, nqa, L.kring, row, S.attn_ws, n, m.heads, row, a.kv_rank, L.ring, m.window, m.scale, c.max_seq_len, pos0, ctl,
+		                                  L.sink, st));
+	else
+		ST_TRY(yalm_attn_window_pool_sink(S.scan, nl, S.aux, nqa, L.kring, row, L.kring, row, nullptr, nullptr, S.attn_ws, n, m.heads, 1, row, a.kv_rank, L.ring, 0, m.window,
+		                                  0, m.scale, f32, c.max_seq_len, pos0, ctl, L.sink, 1, st));
+	return yalm_head_linear_gate_rows(S.att, no, S.scan, nl, L.wuv, dt, m.out_gate ? P + L.o_gate : nullptr, ldp, n, m.heads, m.vdim, a.kv_rank, st);
+}
+
+// One parallel block over n rows: h = norm(x); the mixer reads the (token-shifted) h through ONE packed projection, the experts
+// read h itself; x += residual_mult (mixer + experts).  With norms in groups the residual add also forms the next norm (next_norm: its
+// weight, null: nothing to norm), so that a step launches one norm of its own.  What the rows leave for the next call (previous h, convolution tails, matrix states,
 // keys) is written by the ops themselves.
-int Model::stack_layer_parallel(StackScratch &S, const yalm::StackLayer &L, int n, int pos0, const int *ctl, cudaStream_t st) {
+int Model::stack_layer_parallel(StackScratch &S, const yalm::StackLayer &L, const float *next_norm, int n, int pos0, const int *ctl, cudaStream_t st) {
 	const Config &c = *config;
 	const StackSpec &sp = *c.stack;
 	const yalm::LayerSpec &ls = L.spec;
 	const int dt = static_cast<int>(c.weight_dtype), W = sp.width, f32 = c.weight_dtype == DType::F32;
 	const float woff = sp.norm_one_plus ? 1.f : 0.f;
-	const int ldp = ls.proj_width();
+	const int ldp = ls.proj_width(), bf16 = c.weight_dtype == DType::BF16;
 	float *P = S.qkv;
-	const bool fuse = n == 1 && block_fuse_on();
+	const bool grouped = sp.norm_groups > 0;
+	void *h16 = grouped && !f32 && !tc_off() && n >= 32 && W % 8 == 0 ? S.n16 : nullptr; // h as the operand several products read
+	const bool fuse = n == 1 && !grouped && block_fuse_on();
 	const bool branch = !fuse && !branches_off(); // independent sublayers on side streams, see below
-	cudaStream_t se = st, sr = st;                // the experts' and the delta rule's streams
+	cudaStream_t se = st, sr = st;                // the experts' stream; the delta rule's or the shared expert's
 	const FfnSpec &f = ls.ffn;
 	const int nsum = f.kind == FfnSpec::Moe ? f.top : 0;
 	// The experts only need h.  A prompt portion forks them before the projection (its product leaves SMs idle at small widths:
@@ -1043,12 +1192,24 @@ int Model::stack_layer_parallel(StackScratch &S, const yalm::StackLayer &L, int 
 			se = S.side[0];
 			ST_TRY(cudaEventRecord(S.fork[0], st));
 			ST_TRY(cudaStreamWaitEvent(se, S.fork[0], 0));
+			if (f.shared_ff > 0) {
+				sr = S.side[1];
+				ST_TRY(cudaStreamWaitEvent(sr, S.fork[0], 0));
+			}
 		}
 		return 0;
 	};
 	if (fuse && sp.token_shift && gemv_fusable(c, n, W, L.wproj, S.x)) // a decode row: norm, shift and projection as one launch
 		ST_TRY(yalm_gemv_norm_shift(P, S.x, L.wproj, W, ldp, dt, L.norm1, sp.norm_scalar, woff, sp.norm_eps, L.shift, L.hprev, S.xn, pos0, ctl, S.ticket, st));
-	else {
+	else if (grouped) {
+		if (!S.xn_valid) ST_TRY(yalm_group_norm_rows(S.xn, h16, bf16, S.x, nullptr, L.norm1, sp.norm_groups, sp.norm_eps, n, W, st));
+		S.xn_valid = false;
+		if (n > 1) ST_TRY(fork_experts());
+		int ncols = ldp; // rows of the packed projection, without the padding of a row of results
+		if (ls.kind == yalm::MixerKind::Retention) ncols = L.o_gate + ls.ret.heads * ls.ret.vdim;
+		else if (ls.kind == yalm::MixerKind::Attention) ncols = L.o_gate + (ls.mix.head_gate ? ls.mix.heads : 0);
+		ST_TRY(stack_linear_h(*this, c, S.a16, h16, P, ldp, S.xn, W, L.wproj, n, ncols, W, st));
+	} else {
 		ST_TRY(yalm_norm_shift_rows(S.xn, sp.token_shift ? S.hs : nullptr, S.x, L.norm1, sp.norm_scalar, woff, sp.norm_eps, L.shift, L.hprev, n, W, pos0, ctl, st));
 		if (n > 1) ST_TRY(fork_experts());
 		ST_TRY(stack_linear(*this, c, S.a16, P, ldp, sp.token_shift ? S.hs : S.xn, W, L.wproj, n, ldp, W, 1.f, st));
@@ -1062,8 +1223,15 @@ int Model::stack_layer_parallel(StackScratch &S, const yalm::StackLayer &L, int 
 	auto experts = [&]() -> int {
 		if (!nsum) return 0;
 		const int act = f.act == yalm::GluAct::SigmoidScaled ? 2 : f.act == yalm::GluAct::Silu ? YALM_ACT_SILU : YALM_ACT_GELU;
-		ST_TRY(yalm_router_topk_rows(S.ids, S.wts, S.xn, W, L.router, dt, n, f.experts, f.top, W, f.score == yalm::RouterScore::Sigmoid ? 1 : 0,
-		                             f.renormalize ? 1 : 0, f.renorm_eps, f.groups, f.keep_groups, se));
+		if (f.shared_ff > 0) { // beside the routed experts; first, because their prompt route waits on the host
+			void *op = sr == st ? S.a16 : S.a16r;
+			ST_TRY(stack_linear_h(*this, c, op, h16, S.gu, 2 * f.shared_ff, S.xn, W, L.wsgu, n, 2 * f.shared_ff, W, sr));
+			ST_TRY(yalm_glu_act_rows(S.hsh, S.gu, n, f.shared_ff, glu_act_code(f.shared_act), 1.f, 0.f, 0.f, sr));
+			ST_TRY(stack_linear(*this, c, op, S.y2, W, S.hsh, f.shared_ff, L.wsdown, n, W, f.shared_ff, 1.f, sr));
+		}
+		ST_TRY(yalm_router_group_topk_rows(S.ids, S.wts, S.xn, W, L.router, dt, n, f.experts, f.top, W, f.score == yalm::RouterScore::Sigmoid ? 1 : 0,
+		                                   f.renormalize ? 1 : 0, f.renorm_eps, f.groups, f.keep_groups, f.group_top, f.choice_bias ? L.router_bias : nullptr,
+		                                   f.router_scale, se));
 		if (S.moe_gu && !ctl && n * f.top >= 64 && W % 8 == 0 && f.ff % 8 == 0 && !moe_grouped_off())
 			return stack_moe_grouped(S, L, S.xn, se == st ? S.a16 : S.a16e, n, act, se); // waits on the host for the chosen experts
 		ST_TRY(yalm_moe_glu_slots(S.h, S.xn, W, L.wg, L.wu, dt, S.ids, S.wts, n, f.top, f.ff, W, act, f.act_alpha, f.limit, f.up_offset,
@@ -1093,6 +1261,41 @@ int Model::stack_layer_parallel(StackScratch &S, const yalm::StackLayer &L, int 
 		ST_TRY(yalm_gated_group_norm_rows(S.att, inner, S.scan, inner, P, ldp, L.mix_norm, n, inner, q.norm_groups, sp.norm_eps, st));
 		if (fuse && gemv_fusable(c, n, inner, L.wout, S.att)) return yalm_gemv_residual_sum(S.x, S.y1, S.att, L.wout, 1.f, inner, W, dt, nullptr, S.y, nsum, W, S.ticket, st);
 		ST_TRY(stack_linear(*this, c, S.a16, S.y1, W, S.att, inner, L.wout, n, W, inner, 1.f, st));
+	} else if (ls.kind == yalm::MixerKind::LatentAttention) {
+		const int no = ls.mix.heads * ls.mix.vdim;
+		ST_TRY(stack_latent(S, L, P, ldp, n, pos0, ctl, st));
+		ST_TRY(stack_linear(*this, c, S.a16, S.y1, W, S.att, no, L.wo, n, W, no, 1.f, st));
+	} else if (ls.kind == yalm::MixerKind::Retention) {
+		const yalm::RetentionSpec &r = ls.ret;
+		const int hp = r.heads * r.vdim, inter = r.rot.interleaved ? 1 : 0;
+		if (n == 1)
+			ST_TRY(yalm_retention_step(S.att, L.scan_state, P, L.o_q, L.o_k, L.o_v, L.o_gate, L.decay, L.rot_freq, L.rot_mag, r.rot.dims, inter,
+			                           1.0f / sqrtf((float)r.dim), r.heads, r.dim, r.vdim, sp.norm_eps, pos0, ctl, st));
+		else { // the decays and k's factor are the same for every row: row stride 0
+			ST_TRY(yalm_rotate_heads_rows(P + L.o_q, ldp, 2 * r.heads, r.dim, 0, L.rot_freq, L.rot_mag, r.rot.dims, inter, n, pos0, ctl, st));
+			ST_TRY(yalm_state_scan_rows(S.scan, hp, P + L.o_k, ldp, P + L.o_q, ldp, P + L.o_v, ldp, L.decay, 0, 0, L.k_scale, 0, nullptr, 0, nullptr, L.scan_state, n,
+			                            r.heads, 1, r.dim, r.vdim, pos0, ctl, st));
+			ST_TRY(yalm_head_norm_act_rows(S.att, hp, S.scan, hp, P + L.o_gate, ldp, nullptr, n, r.heads, r.vdim, sp.norm_eps, 1, st));
+		}
+		ST_TRY(stack_linear(*this, c, S.a16, S.y1, W, S.att, hp, L.wo, n, W, hp, 1.f, st));
+	} else if (ls.kind == yalm::MixerKind::Attention) {
+		const yalm::MixerSpec &m = ls.mix;
+		const int no = m.heads * m.vdim;
+		ST_TRY(yalm_qkv_bias_post_rows(P, ldp, L.qkb, L.kring, L.vring, nullptr, 0, L.qnorm, L.knorm, nullptr, 0, n, m.heads, m.kv_heads, m.dim, m.vdim, L.ring,
+		                               sp.norm_eps, f32, pos0, ctl, st));
+		const float *gate = m.head_gate ? P + L.o_gate : nullptr;
+		const float *Q = P + L.o_q;
+		// prompt portions and decode rows over bf16 rings: tensor cores; the fp32 rings and other sizes: the SIMT kernel
+		if (!f32 && n >= 16 && ldp % 4 == 0 && yalm_attn_mixed_mma_shape(m.heads, m.kv_heads, m.dim, m.vdim) && !attn_mma_off())
+			ST_TRY(yalm_attn_mixed_mma(S.att, no, Q, ldp, L.kring, L.vring, L.bias_table, L.n_bias, L.talk, gate, ldp, S.mixed_ws, S.mixed_floats, n, m.heads, m.kv_heads,
+			                           m.dim, m.vdim, L.ring, m.window, m.scale, m.softcap, c.max_seq_len, pos0, ctl, st));
+		else if (!f32 && ldp % 4 == 0 && yalm_attn_mixed_decode_shape(m.heads, m.kv_heads, m.dim, m.vdim) && !attn_mma_off())
+			ST_TRY(yalm_attn_mixed_decode(S.att, no, Q, ldp, L.kring, L.vring, L.bias_table, L.n_bias, L.talk, gate, ldp, S.mixed_ws, S.mixed_floats, n, m.heads,
+			                              m.kv_heads, m.dim, m.vdim, L.ring, m.window, m.scale, m.softcap, c.max_seq_len, pos0, ctl, st));
+		else
+			ST_TRY(yalm_attn_mixed_rows(S.att, no, Q, ldp, L.kring, L.vring, L.bias_table, L.n_bias, L.talk, gate, ldp, S.mixed_ws, S.mixed_floats, n, m.heads, m.kv_heads,
+			                            m.dim, m.vdim, L.ring, m.window, m.scale, m.softcap, f32, c.max_seq_len, pos0, ctl, st));
+		ST_TRY(stack_linear(*this, c, S.a16, S.y1, W, S.att, no, L.wo, n, W, no, 1.f, st));
 	} else {
 		if (branch) {
 			sr = S.side[1];
@@ -1130,11 +1333,13 @@ int Model::stack_layer_parallel(StackScratch &S, const yalm::StackLayer &L, int 
 	}
 	if (branch) ST_TRY(experts()); // enqueued last: its host wait (prompt portions) then overlaps the mixer's kernels
 	ST_TRY(join());
+	if (grouped) {
+		ST_TRY(yalm_residual_group_norm_rows(S.x, sp.residual_mult, S.y1, L.o_bias, f.shared_ff > 0 ? S.y2 : nullptr, nsum ? S.y : nullptr, W, nsum,
+		                                     next_norm ? S.xn : nullptr, next_norm ? h16 : nullptr, bf16, next_norm, sp.norm_groups, sp.norm_eps, n, W, st));
+		S.xn_valid = next_norm != nullptr;
+		return 0;
+	}
 	return yalm_residual_sum_rows(S.x, S.y1, mix_b, S.y, W, nsum, n, W, st);
-}
-
-static int glu_act_code(yalm::GluAct a) {
-	return a == yalm::GluAct::SigmoidScaled ? 2 : a == yalm::GluAct::GeluTanh ? 3 : a == yalm::GluAct::Silu ? YALM_ACT_SILU : YALM_ACT_GELU;
 }
 
 // One pre-norm layer over n rows: u = N1(x) + conv(N1(x)), x += mixer(u); v = N2(x) + conv(N2(x)), x += ff(v); then the
@@ -1145,48 +1350,15 @@ int Model::stack_layer_prenorm(StackScratch &S, const yalm::StackLayer &L, int i
 	const Config &c = *config;
 	const StackSpec &sp = *c.stack;
 	const yalm::LayerSpec &ls = L.spec;
-	const int dt = static_cast<int>(c.weight_dtype), W = sp.width, f32 = c.weight_dtype == DType::F32, taps = std::max(1, sp.input_conv);
+	const int dt = static_cast<int>(c.weight_dtype), W = sp.width, taps = std::max(1, sp.input_conv);
 	const int ldp = ls.proj_width();
 	float *P = S.qkv;
 	// ---- token mixer ----
 	ST_TRY(yalm_norm_conv_rows(S.hs, S.xn, S.x, L.norm1, sp.layer_norm ? 1 : 0, sp.norm_eps, L.inconv1, L.inconv1_state, n, W, taps, pos0, ctl, st));
 	ST_TRY(stack_linear(*this, c, S.a16, P, ldp, S.hs, W, L.wproj, n, ldp, W, 1.f, st));
 	if (ls.kind == yalm::MixerKind::LatentAttention) {
-		const yalm::MixerSpec &m = ls.mix;
-		const yalm::LatentSpec &a = ls.latent;
-		const int row = a.kv_rank + a.rot_dim, nq = m.heads * (m.dim + a.rot_dim), nqa = m.heads * row, nl = m.heads * a.kv_rank, no = m.heads * m.vdim;
-		const bool own = a.kv_from < 0;
-		ST_TRY(yalm_latent_post_rows(P, ldp, L.o_q, a.q_rank, L.qnorm, L.o_kv, a.kv_rank, a.rot_dim, L.knorm, own ? L.kring : nullptr, L.ring, L.rot_freq,
-		                             L.rot_mag, a.rot.dims, a.rot.interleaved ? 1 : 0, sp.norm_eps, f32, n, pos0, ctl, st));
-		ST_TRY(stack_linear(*this, c, S.a16, S.conv, nq, P + L.o_q, ldp, L.wuq, n, nq, a.q_rank, 1.f, st));
-		const int dk = m.dim + a.rot_dim;
-		if (!f32 && !ctl && n >= 16 && m.window > 0 && m.dim > 0 && S.lat16 && a.kv_rank % 8 == 0 && nq % 4 == 0 && no % 2 == 0 && (m.heads * (m.dim + m.vdim)) % 4 == 0 &&
-		    yalm_attn_window_pool_mma_shape(dk, m.vdim) && !attn_mma_off()) {
-			// A prompt portion in 16-bit: the latents of the visible rows times [W_uk ; W_uv] on the tensor cores give every head's keys
-			// and values, written beside the rotated key part into head-major rings for the windowed tensor-core attention; the queries
-			// stay as projected, their rotated part turned in place.
-			const int first = std::max(0, pos0 - m.window + 1), count = pos0 + n - first, nkv = m.heads * (m.dim + m.vdim);
-			ST_TRY(yalm_latent_gather_rows16(S.lat16, L.kring, L.ring, row, a.kv_rank, first, count, st));
-			ST_TRY(yalm_gemm_16(S.latkv, nkv, S.lat16, L.wuk, count, nkv, a.kv_rank, 0, dt == YALM_BF16, 1.f, st));
-			ST_TRY(yalm_latent_pack_rings(S.lat_ek, S.lat_ev, S.latkv, nkv, L.kring, L.ring, a.kv_rank, a.rot_dim, m.heads, m.dim, m.vdim, L.ring, first, count, st));
-			ST_TRY(yalm_rotate_heads_rows(S.conv, nq, m.heads, dk, m.dim, L.rot_freq, L.rot_mag, a.rot.dims, a.rot.interleaved ? 1 : 0, n, pos0, ctl, st));
-			ST_TRY(yalm_attn_window_pool_mma(S.att, no, S.conv, nq, S.lat_ek, S.lat_ev, nullptr, nullptr, n, m.heads, m.heads, dk, m.vdim, L.ring, 0, m.window, 0,
-			                                 m.scale, pos0, ctl, st));
-			if (m.out_gate) ST_TRY(yalm_sigmoid_gate_rows(S.att, no, P + L.o_gate, ldp, n, no, st));
-		} else {
-			// A decode row (and what the tensor-core route does not take): W_uk moves to the query side, every head reads the one cached
-			// row of a position — keys are whole rows, values their first kv_rank channels — and W_uv follows the weighted sum.
-			ST_TRY(yalm_latent_query_rows(S.aux, nqa, S.conv, nq, L.wukt, dt, n, m.heads, m.dim, a.rot_dim, a.kv_rank, L.rot_freq, L.rot_mag, a.rot.dims,
-			                              a.rot.interleaved ? 1 : 0, pos0, ctl, st));
-			static const bool one_pass_off = [] { const char *e = getenv("YALM_STACK_ATTN_LANES"); return e && e[0] == '0'; }();
-			if (!f32 && !one_pass_off && yalm_attn_latent_rows_shape(row, a.kv_rank, row) && ((uintptr_t)L.kring & 15) == 0 && nqa % 4 == 0)
-				ST_TRY(yalm_attn_latent_rows(S.scan, nl, S.aux, nqa, L.kring, row, S.attn_ws, n, m.heads, row, a.kv_rank, L.ring, m.window, m.scale, c.max_seq_len,
-				                             pos0, ctl, st));
-			else
-				ST_TRY(yalm_attn_window_pool_strided(S.scan, nl, S.aux, nqa, L.kring, row, L.kring, row, nullptr, nullptr, S.attn_ws, n, m.heads, 1, row, a.kv_rank,
-				                                     L.ring, 0, m.window, 0, m.scale, f32, c.max_seq_len, pos0, ctl, st));
-			ST_TRY(yalm_head_linear_gate_rows(S.att, no, S.scan, nl, L.wuv, dt, m.out_gate ? P + L.o_gate : nullptr, ldp, n, m.heads, m.vdim, a.kv_rank, st));
-		}
+		const int no = ls.mix.heads * ls.mix.vdim;
+		ST_TRY(stack_latent(S, L, P, ldp, n, pos0, ctl, st));
 		ST_TRY(stack_linear(*this, c, S.a16, S.y1, W, S.att, no, L.wo, n, W, no, 1.f, st));
 	} else {
 		const yalm::GlaSpec &g = ls.gla;
@@ -1378,46 +1550,8 @@ int Model::stack_layer_sandwich(StackScratch &S, const yalm::StackLayer &L, cons
 	if (!S.xn_valid) ST_TRY(yalm_norm_shift_rows(S.xn, nullptr, S.x, L.norm1, 0, 0.f, sp.norm_eps, nullptr, nullptr, n, W, pos0, ctl, st));
 	S.xn_valid = false;
 	if (ls.kind == yalm::MixerKind::LatentAttention) {
-		const yalm::LatentSpec &a = ls.latent;
-		const int row = a.kv_rank + a.rot_dim, nqa = m.heads * row, nl = m.heads * a.kv_rank, dk = m.dim + a.rot_dim;
-		const bool own = a.kv_from < 0;
 		ST_TRY(stack_linear(*this, c, S.a16, P, ldp, S.xn, W, L.wproj, n, ldp, W, 1.f, st));
-		if (own)
-			ST_TRY(yalm_latent_post_rows(P, ldp, L.o_q, 0, nullptr, L.o_kv, a.kv_rank, a.rot_dim, L.knorm, L.kring, L.ring, L.rot_freq, L.rot_mag, a.rot.dims,
-			                             a.rot.interleaved ? 1 : 0, sp.norm_eps, f32, n, pos0, ctl, st));
-		float *Q = P + L.o_q; // the queries as projected, per head [unrotated | rotated part]
-		if (!f32 && !ctl && n >= 16 && m.dim > 0 && S.lat16 && a.kv_rank % 8 == 0 && ldp % 4 == 0 && no % 2 == 0 && (m.heads * (m.dim + m.vdim)) % 4 == 0 &&
-		    yalm_attn_window_pool_mma_shape(dk, m.vdim) && !attn_mma_off()) {
-			// A prompt portion in 16-bit: the latents of the visible rows times [W_uk ; W_uv] on the tensor cores give every head's keys
-			// and values, written beside the rotated key part into head-major rings for the tensor-core attention.
-			const int first = m.window > 0 ? std::max(0, pos0 - m.window + 1) : 0, count = pos0 + n - first, nkv = m.heads * (m.dim + m.vdim);
-			ST_TRY(yalm_latent_gather_rows16(S.lat16, L.kring, L.ring, row, a.kv_rank, first, count, st));
-			ST_TRY(yalm_gemm_16(S.latkv, nkv, S.lat16, L.wuk, count, nkv, a.kv_rank, 0, dt == YALM_BF16, 1.f, st));
-			ST_TRY(yalm_latent_pack_rings(S.lat_ek, S.lat_ev, S.latkv, nkv, L.kring, L.ring, a.kv_rank, a.rot_dim, m.heads, m.dim, m.vdim, L.ring, first, count, st));
-			ST_TRY(yalm_rotate_heads_rows(Q, ldp, m.heads, dk, m.dim, L.rot_freq, L.rot_mag, a.rot.dims, a.rot.interleaved ? 1 : 0, n, pos0, ctl, st));
-			ST_TRY(yalm_attn_window_pool_mma_sink(S.att, no, Q, ldp, S.lat_ek, S.lat_ev, nullptr, nullptr, n, m.heads, m.heads, dk, m.vdim, L.ring, 0, m.window, 0,
-			                                      m.scale, pos0, ctl, L.sink, m.heads, st));
-		} else {
-			// A decode row (and what the tensor-core route does not take): W_uk moves to the query side, every head reads the one cached
-			// row of a position — keys are whole rows, values their first kv_rank channels — and W_uv follows the weighted sum.
-			ST_TRY(yalm_latent_query_rows(S.aux, nqa, Q, ldp, L.wukt, dt, n, m.heads, m.dim, a.rot_dim, a.kv_rank, L.rot_freq, L.rot_mag, a.rot.dims,
-			                              a.rot.interleaved ? 1 : 0, pos0, ctl, st));
-			static const bool latent_mma_off = [] { const char *e = getenv("YALM_STACK_LATENT_MMA"); return e && e[0] == '0'; }(); // A/B against the SIMT kernel
-			if (!f32 && !latent_mma_off && yalm_attn_latent_mma_shape(row, a.kv_rank, row) && ((uintptr_t)L.kring & 15) == 0 && nqa % 4 == 0 && n * m.heads <= 4096) {
-				// the heads as the M tile of the tensor cores; the keys a row can ever see, in tiles of 64, are split over up to 128 CTAs (shapes only)
-				const int tiles = ((m.window > 0 ? std::min(m.window, c.max_seq_len) : c.max_seq_len) + 63) / 64, ctas = (m.heads + 15) / 16 * n;
-				const int cap = std::max(1, std::min({tiles, 128, 4096 / (n * m.heads), (296 + ctas - 1) / ctas}));
-				const int per = (tiles + cap - 1) / cap, nsplit = (tiles + per - 1) / per;
-				ST_TRY(yalm_attn_latent_mma_rows(S.scan, nl, S.aux, nqa, L.kring, row, S.attn_ws, n, m.heads, row, a.kv_rank, L.ring, m.window, m.scale, nsplit, pos0,
-				                                 ctl, L.sink, st));
-			} else if (!f32 && yalm_attn_latent_rows_shape(row, a.kv_rank, row) && ((uintptr_t)L.kring & 15) == 0 && nqa % 4 == 0)
-				ST_TRY(yalm_attn_latent_rows_sink(S.scan, nl, S.aux, nqa, L.kring, row, S.attn_ws, n, m.heads, row, a.kv_rank, L.ring, m.window, m.scale,
-				                                  c.max_seq_len, pos0, ctl, L.sink, st));
-			else
-				ST_TRY(yalm_attn_window_pool_sink(S.scan, nl, S.aux, nqa, L.kring, row, L.kring, row, nullptr, nullptr, S.attn_ws, n, m.heads, 1, row, a.kv_rank,
-				                                  L.ring, 0, m.window, 0, m.scale, f32, c.max_seq_len, pos0, ctl, L.sink, 1, st));
-			ST_TRY(yalm_head_linear_gate_rows(S.att, no, S.scan, nl, L.wuv, dt, nullptr, 0, n, m.heads, m.vdim, a.kv_rank, st));
-		}
+		ST_TRY(stack_latent(S, L, P, ldp, n, pos0, ctl, st));
 	} else {
 		const int nqv = m.maps * m.heads, nkv = m.maps * m.kv_heads, ncols = L.o_gate + (m.head_gate ? m.heads : 0), na = m.maps * no;
 		const int keep = L.max_blocks, pool = keep > 0 ? 1 : 0;
@@ -1529,7 +1663,8 @@ int Model::stack_pass(InferenceState &s, int n, int pos0, bool from_ctl, int n_w
 			continue;
 		}
 		if (sp.parallel_block) {
-			ST_TRY(stack_layer_parallel(S, L, n, pos0, ctl, st));
+			// what the residual add may norm next: the following layer's input or, for a decode row, the head's
+			ST_TRY(stack_layer_parallel(S, L, li + 1 < _stack.size() ? _stack[li + 1]->norm1 : n == 1 && n_want == 1 ? rms_final_weight : nullptr, n, pos0, ctl, st));
 			ST_TRY(tap());
 			continue;
 		}
@@ -1599,7 +1734,9 @@ int Model::stack_pass(InferenceState &s, int n, int pos0, bool from_ctl, int n_w
 	if (n_want > 0) {
 		if (sp.norm_bias && n_want == 1 && sp.logit_scale == 1.f && !(sp.logit_softcap > 0.f) && gemv_fusable(c, n, W, wcls, S.x)) // a decode row: norm + head as one launch
 			return yalm_gemv_block_in(s.logits_dev(), S.x, wcls, W, sp.vocab, dt, rms_final_weight, _final_bias, sp.norm_eps, 1, nullptr, nullptr, 1, nullptr, pos0, ctl, st);
-		if (sp.norm_bias)
+		if (sp.norm_groups > 0) {
+			if (!S.xn_valid) ST_TRY(yalm_group_norm_rows(S.xn, nullptr, 0, S.x, from_ctl ? nullptr : S.want, rms_final_weight, sp.norm_groups, sp.norm_eps, n_want, W, st));
+		} else if (sp.norm_bias)
 			ST_TRY(yalm_layer_norm_rows(S.xn, nullptr, 0, S.x, nullptr, from_ctl ? nullptr : S.want, rms_final_weight, _final_bias, sp.norm_eps, n_want, W, st));
 		else if (sp.layer_norm)
 			ST_TRY(yalm_layer_norm_gather_rows(S.xn, S.x, from_ctl ? nullptr : S.want, rms_final_weight, 1, sp.norm_eps, n_want, W, st));

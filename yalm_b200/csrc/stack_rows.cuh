@@ -123,38 +123,56 @@ __device__ __forceinline__ float act_value(float z, int act) {
 	return act_gelu(z);
 }
 
+// ---- rotary positions ---------------------------------------------------------------------------------------------------
+// Pair i of a vector at position p turns by p * freq[i]; cos and sin carry the magnitude factor.  Position, angle and the
+// rotation are fp32.  interleaved: the pair is (2 i, 2 i + 1), else (i, i + half).
+__device__ __forceinline__ void rotate_pair(float a, float b, int p, float freq, float mag, float *ra, float *rb) {
+	const float ang = (float)p * freq;
+	float sn, cs;
+	sincosf(ang, &sn, &cs);
+	sn *= mag, cs *= mag;
+	*ra = a * cs - b * sn, *rb = b * cs + a * sn;
+}
+
 // Row `row` of q | k | v (fp32) at ring slot `slot`: RMS norm over the WHOLE q and k projections (all heads at once), one
 // weight per channel (qnorm / knorm null: left as they are); q stays in place, k goes to the ring.  v: vmode 1 keeps a copy
 // in vfirst (the first blending layer), vmode 2 blends v = (1 - lambda) v + lambda vfirst (later blending layers); the
 // blended v is what is cached.  Caches are head-major (kv head, slot, channel).  All threads of the CTA take part.  The row
-// is read past L1 (__ldcg): in the fused tail other CTAs of the same launch wrote it.
+// is read past L1 (__ldcg): in the fused tail other CTAs of the same launch wrote it.  bias (q | k | v; null: none) is added first.
 template <typename CT>
 __device__ __forceinline__ void qkv_post_row(float *row, CT *kc, CT *vc, float *vfirst, const float *qnorm, const float *knorm, const float *vmix, int vmode,
-                                             int nq, int nk, int nv, int dk, int dv, int ring, int slot, float eps, float *red) {
+                                             int nq, int nk, int nv, int dk, int dv, int ring, int slot, float eps, float *red, const float *bias = nullptr) {
+	auto in = [&](int e) { return bias ? __ldcg(row + e) + bias[e] : __ldcg(row + e); };
 	float rq = 1.f, rk = 1.f;
 	if (qnorm) {
 		float s = 0.f;
-		for (int e = threadIdx.x; e < nq; e += blockDim.x) s += __ldcg(row + e) * __ldcg(row + e);
+		for (int e = threadIdx.x; e < nq; e += blockDim.x) {
+			const float v = in(e);
+			s += v * v;
+		}
 		s = block_sum(s, red);
 		rq = 1.0f / sqrtf(s / nq + eps);
 	}
 	if (knorm) {
 		float s = 0.f;
-		for (int e = threadIdx.x; e < nk; e += blockDim.x) s += __ldcg(row + nq + e) * __ldcg(row + nq + e);
+		for (int e = threadIdx.x; e < nk; e += blockDim.x) {
+			const float v = in(nq + e);
+			s += v * v;
+		}
 		s = block_sum(s, red);
 		rk = 1.0f / sqrtf(s / nk + eps);
 	}
-	if (qnorm)
-		for (int e = threadIdx.x; e < nq; e += blockDim.x) row[e] = __ldcg(row + e) * rq * qnorm[e];
+	if (qnorm || bias)
+		for (int e = threadIdx.x; e < nq; e += blockDim.x) row[e] = qnorm ? in(e) * rq * qnorm[e] : in(e);
 	for (int e = threadIdx.x; e < nk; e += blockDim.x) {
-		float v = __ldcg(row + nq + e);
+		float v = in(nq + e);
 		if (knorm) v = v * rk * knorm[e];
 		const int g = e / dk, d = e % dk;
 		cache_put(kc, ((size_t)g * ring + slot) * dk + d, v);
 	}
 	const float lam = vmode == 2 ? vmix[0] : 0.f;
 	for (int e = threadIdx.x; e < nv; e += blockDim.x) {
-		float v = __ldcg(row + nq + nk + e);
+		float v = in(nq + nk + e);
 		if (vmode == 1) vfirst[e] = v;
 		else if (vmode == 2) v = (1.0f - lam) * v + lam * vfirst[e];
 		const int g = e / dv, d = e % dv;

@@ -340,7 +340,8 @@ private:
 	               float *probs_out);
 	int stack_pass(InferenceState &s, int n, int pos0, bool from_ctl, int n_want);
 	int stack_moe_grouped(StackScratch &S, const yalm::StackLayer &L, const float *x, void *a16, int n, int act, cudaStream_t st);
-	int stack_layer_parallel(StackScratch &S, const yalm::StackLayer &L, int n, int pos0, const int *ctl, cudaStream_t st);
+	int stack_latent(StackScratch &S, const yalm::StackLayer &L, float *P, int ldp, int n, int pos0, const int *ctl, cudaStream_t st);
+	int stack_layer_parallel(StackScratch &S, const yalm::StackLayer &L, const float *next_norm, int n, int pos0, const int *ctl, cudaStream_t st);
 	int stack_layer_block(StackScratch &S, const yalm::StackLayer &L, const yalm::StackLayer *next, int n, int pos0, const int *ctl, cudaStream_t st);
 	int stack_layer_prenorm(StackScratch &S, const yalm::StackLayer &L, int index, int n, int pos0, const int *ctl, cudaStream_t st);
 	int stack_layer_sandwich(StackScratch &S, const yalm::StackLayer &L, const yalm::StackLayer *next, int index, int n, int pos0, const int *ctl, bool from_ctl,
