@@ -51,6 +51,7 @@ WORKLOADS = {
     "fegizen-sizes": ("tiny", "bf16", 4096, "Fegizen (latent attention over cached latents / gated linear attention, experts with identity and shared experts) at model-like sizes"),
     "kiduvik-sizes": ("tiny", "bf16", 4096, "Kiduvik (latent attention with a sink over cached latents / differential attention over a window with kept first tokens, dense feed-forward, token side input) at model-like sizes"),
     "fafelix-sizes": ("tiny", "bf16", 4096, "Fafelix (parallel blocks: gated delta rule / causal attention with a sink / time mixing, dense feed-forward, repeated layer spans) at model-like sizes"),
+    "desalorn-sizes": ("tiny", "bf16", 4096, "Desalorn (parallel blocks: attention with mixed head scores / retention / windowed latent attention, routed experts over groups and a shared one) at model-like sizes"),
     "mistral-7b-fp16-prefill": ("mistral-7b", "fp16", 4096, "Mistral-7B-v0.2 fp16 random-init, 4096-token prompt hydrated in 512-token chunks (tcgen05 GEMMs)"),
 }
 HEADLINE = "mistral-7b-fp16-4k"
@@ -386,6 +387,11 @@ def main():
             raise SystemExit("bench.py: the layered models run on one GPU")
         from yalm_b200 import stack_bench
         return stack_bench.run_fafelix(args, base, _emit, shm_path, ClockSampler)
+    if args.workload == "desalorn-sizes":
+        if world > 1:
+            raise SystemExit("bench.py: the layered models run on one GPU")
+        from yalm_b200 import stack_bench
+        return stack_bench.run_desalorn(args, base, _emit, shm_path, ClockSampler)
     if args.workload.endswith("-prefill"):
         if world > 1:
             raise SystemExit("bench.py: the prefill workload is single-GPU")

@@ -752,6 +752,163 @@ def run_fafelix(args, base, emit, shm_path, ClockSampler):
                           l2="inputs larger than L2 (weights streamed per token)")))
 
 
+# ---- Desalorn --------------------------------------------------------------------------------------------------------------
+# name: width; attention heads / kv heads / head size, distance table rows and farthest distance; latent attention heads x (dim unrotated +
+# rot rotated) keys, vdim values, latent sizes, window; retention heads x (dim, vdim); experts (groups, shared expert); layer order
+# (l = latent attention, a = attention with mixed head scores, r = retention), every layer with experts
+DESALORN_SIZES = {
+    "w1024": dict(width=1024, heads=8, kv_heads=2, dim=128, rel=32, far=512, lheads=8, ldim=64, rot=64, lvdim=128, kv_rank=256, q_rank=512, window=1024, rheads=8, rdim=128,
+                  rvdim=128, moe_ff=1024, experts=8, top=2, groups=4, keep_groups=2, shared=1024, order="larl", vocab=32000),
+    "w2048": dict(width=2048, heads=16, kv_heads=4, dim=128, rel=32, far=512, lheads=16, ldim=64, rot=64, lvdim=128, kv_rank=512, q_rank=1024, window=1024, rheads=16, rdim=128,
+                  rvdim=128, moe_ff=2048, experts=8, top=2, groups=4, keep_groups=2, shared=2048, order="larl", vocab=32000),
+}
+
+
+def write_desalorn(folder, z):
+    """A checkpoint directory of the given size: matrices tiled from one random block, norm weights 1."""
+    os.makedirs(folder, exist_ok=True)
+    rng = np.random.default_rng(6)
+    block = _bf16(rng.standard_normal(1 << 22).astype(np.float32) * 0.02)
+    W = z["width"]
+    mlp = {"kind": "moe", "expert": {"ff": z["moe_ff"]}, "router": {"experts": z["experts"], "top": z["top"], "groups": {"count": z["groups"], "keep": z["keep_groups"]}},
+           "shared": {"ff": z["shared"]}}
+    mixers = {"a": ("attention", {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["dim"], "scale": z["dim"] ** -0.5, "softcap": 30.0, "bias_max": z["far"]}),
+              "l": ("latent_attention", {"heads": z["lheads"], "dim": z["ldim"], "rot_dim": z["rot"], "vdim": z["lvdim"], "kv_rank": z["kv_rank"], "q_rank": z["q_rank"],
+                                         "mask": {"size": z["window"]}, "rot": {"base": 10000.0, "dims": z["rot"]}, "scale": (z["ldim"] + z["rot"]) ** -0.5}),
+              "r": ("retention", {"heads": z["rheads"], "dim": z["rdim"], "vdim": z["rvdim"], "rot": {"base": 10000.0, "dims": z["rdim"]},
+                                  "decay": [1.0 - 2.0 ** (-5 - 3.0 * i / z["rheads"]) for i in range(z["rheads"])]})}
+    cfg = {"architecture": "Desalorn", "width": W, "vocab": z["vocab"], "norm": {"eps": 1e-5, "groups": 2}, "embedding": {"scale": 1.0}, "residual_mult": 0.5,
+           "layers": [{"type": mixers[c][0], "mixer": mixers[c][1], "mlp": mlp} for c in z["order"]]}
+    with open(os.path.join(folder, "config.json"), "w") as f:
+        json.dump(cfg, f)
+    shapes = {"embed": (z["vocab"], W), "final.norm": (W,), "head": (z["vocab"], W)}
+    for i, c in enumerate(z["order"]):
+        p, m, f = "l%d." % i, "l%d.mix." % i, "l%d.mlp." % i
+        shapes.update({p + "norm1": (W,), f + "router": (z["experts"], W), f + "correction": (z["experts"],)})
+        for e in ["e%d." % e for e in range(z["experts"])] + ["shared."]:
+            ff = z["shared"] if e == "shared." else z["moe_ff"]
+            shapes.update({f + e + "gate": (ff, W), f + e + "up": (ff, W), f + e + "down": (W, ff)})
+        if c == "a":
+            H, nq, nk = z["heads"], z["heads"] * z["dim"], z["kv_heads"] * z["dim"]
+            shapes.update({m + "q": (nq, W), m + "q.b": (nq,), m + "k": (nk, W), m + "k.b": (nk,), m + "v": (nk, W), m + "v.b": (nk,), m + "q.norm": (nq,), m + "k.norm": (nk,),
+                           m + "rel": (z["rel"], H), m + "talk": (H, H), m + "g": (H, W), m + "o": (W, nq), m + "o.b": (W,)})
+        elif c == "l":
+            H, no = z["lheads"], z["lheads"] * z["lvdim"]
+            shapes.update({m + "dq": (z["q_rank"], W), m + "dq.norm": (z["q_rank"],), m + "uq": (H * (z["ldim"] + z["rot"]), z["q_rank"]),
+                           m + "dkv": (z["kv_rank"] + z["rot"], W), m + "dkv.norm": (z["kv_rank"],), m + "uk": (H * z["ldim"], z["kv_rank"]), m + "uv": (no, z["kv_rank"]),
+                           m + "o": (W, no)})
+        else:
+            hd, hp = z["rheads"] * z["rdim"], z["rheads"] * z["rvdim"]
+            shapes.update({m + "q": (hd, W), m + "k": (hd, W), m + "v": (hp, W), m + "g": (hp, W), m + "o": (W, hp)})
+    header, off = {}, 0
+    for name, shp in shapes.items():
+        n = int(np.prod(shp))
+        header[name] = {"dtype": "BF16", "shape": list(shp), "data_offsets": [off, off + 2 * n]}
+        off += 2 * n
+    h = json.dumps(header).encode()
+    h += b" " * (-len(h) % 8)
+    one = _bf16(np.ones(1, np.float32))[0]
+    with open(os.path.join(folder, "model.safetensors"), "wb") as f:
+        f.write(struct.pack("<Q", len(h)) + h)
+        for k, (name, shp) in enumerate(shapes.items()):
+            n = int(np.prod(shp))
+            if name.endswith("norm") or name.endswith("norm1"):
+                f.write(np.full(n, one, np.uint16).tobytes())
+            elif len(shp) < 2:
+                f.write(block[:n].tobytes())
+            else:
+                f.write(np.resize(np.roll(block, 7919 * k), n).tobytes())
+    return cfg
+
+
+def desalorn_numbers(z):
+    """-> (decode bytes per token at CONTEXT, prefill FLOP per token): the active matrices once (bf16), the fp32 matrix states read and
+    written, all earlier keys and values of the attention layers, the window of cached latents; 2 FLOP per active parameter plus the
+    attentions' products (over the causal half of the context or the window; the mixing: 2 heads^2 per key) and the recurrence's own."""
+    W, H = z["width"], z["heads"]
+    experts = (z["top"] * 3 * z["moe_ff"] + z["experts"] + 3 * z["shared"]) * W
+    params, state, extra = z["vocab"] * W, 0, 0.0
+    for c in z["order"]:
+        params += experts
+        if c == "a":
+            nq, nk = H * z["dim"], z["kv_heads"] * z["dim"]
+            params += (2 * nq + 2 * nk + H) * W
+            state += CONTEXT * 2 * nk * 2
+            extra += (4.0 * nq + 2.0 * H * H) * CONTEXT / 2
+        elif c == "l":
+            h, no, row, seen = z["lheads"], z["lheads"] * z["lvdim"], z["kv_rank"] + z["rot"], min(CONTEXT, z["window"])
+            params += (z["q_rank"] + row + no) * W + h * (z["ldim"] + z["rot"]) * z["q_rank"] + h * z["ldim"] * z["kv_rank"] + no * z["kv_rank"]
+            state += seen * row * 2
+            extra += 2.0 * h * (z["ldim"] + z["rot"] + z["lvdim"]) * seen
+        else:
+            hd, hp = z["rheads"] * z["rdim"], z["rheads"] * z["rvdim"]
+            params += (2 * hd + 3 * hp) * W
+            state += 2 * 4 * z["rheads"] * z["rdim"] * z["rvdim"]
+            extra += 6.0 * z["rheads"] * z["rdim"] * z["rvdim"]
+    return 2 * params + state, 2.0 * (params - z["vocab"] * W) + extra
+
+
+def run_desalorn(args, base, emit, shm_path, ClockSampler):
+    """`bench.py --workload desalorn-sizes`: the Desalorn design beside the closest existing models on the same executor: Fegizen (windowed
+    latent attention, a matrix-state recurrence, routed experts and a shared one) and Fapudra (parallel blocks, attention with a
+    distance bias, experts over groups), at equal width, heads, experts, layers and vocabulary."""
+    import torch
+    from yalm_b200 import api
+    pk = os.path.join(ROOT, "MEASURED_PEAKS.json")
+    peaks = json.load(open(pk)) if os.path.exists(pk) else {"hbm_gbs": 6650.0, "bf16_tflops_sustained": 1400.0}
+    hbm, tflops = float(peaks["hbm_gbs"]), float(peaks["bf16_tflops_sustained"])
+    steps = max(8, min(args.steps, 128))
+    clocks = ClockSampler(0)
+    clocks.start()
+    out, launches = [], 0
+
+    def line(write, context, numbers, ids):
+        folder = shm_path("yalm_bench_desalorn_%d" % os.getpid())
+        try:
+            write(folder)
+            model = api.Model(folder, context, api.BF16).cuda(0)
+        finally:
+            shutil.rmtree(folder, ignore_errors=True)
+        st = api.InferenceState(model)
+        st.forward_batch(ids[:1024], 0)                     # warm-up (sizes kernels, first-use set-up)
+        st.end_sequence()
+        torch.cuda.synchronize()
+        t0 = time.perf_counter()
+        st.forward_batch(ids[:-1], 0)
+        t_pre = time.perf_counter() - t0
+        st.generate_greedy(ids[-1], CONTEXT - 1, max(3, args.warmup))   # first step eager + graph capture, untimed
+        st.generate_greedy(ids[0], CONTEXT - 1 + max(3, args.warmup), steps)
+        pre, dec, n = (CONTEXT - 1) / t_pre, steps / (st.device_ms / 1e3), model.launches()
+        st.close()
+        model.close()
+        dec_bytes, pre_flop = numbers
+        return {"prefill_tok_s": pre, "decode_tok_s": dec, "prefill_frac_of_measured_bf16": pre_flop * pre / 1e12 / tflops,
+                "decode_frac_of_measured_hbm": dec_bytes * dec / 1e9 / hbm, "decode_bytes_per_token": dec_bytes, "launches_per_token": n}
+
+    only = os.environ.get("YALM_BENCH_SIZES", "").split(",") if os.environ.get("YALM_BENCH_SIZES") else None
+    ctx = CONTEXT + steps + args.warmup + 8
+    for name, z in DESALORN_SIZES.items():
+        if only and name not in only:
+            continue
+        ids = [(i * 7919 + 1) % z["vocab"] for i in range(CONTEXT)]
+        row = {"size": name, "width": z["width"], "layers": z["order"], "context": CONTEXT, "window": z["window"]}
+        row["desalorn"] = line(lambda f: write_desalorn(f, z), ctx, desalorn_numbers(z), ids)
+        launches += steps * row["desalorn"]["launches_per_token"]
+        if not os.environ.get("YALM_BENCH_NO_PEER"):
+            zg, zf = FEGIZEN_SIZES[name], FAPUDRA_SIZES[name]
+            row["equal_size_fegizen"] = line(lambda f: write_fegizen(f, zg), ctx, fegizen_numbers(zg), ids)
+            row["equal_size_fapudra"] = line(lambda f: write_fapudra(f, zf, ctx), 0, fapudra_numbers(zf), ids)
+        out.append(row)
+    clk = clocks.stop()
+    first = out[0]["desalorn"]
+    emit(dict(base, impl="ours", metric="batch-1 decode tok/s (Desalorn, first size; all sizes under `sizes`)", value=first["decode_tok_s"], steps=steps,
+              ms_per_step=1000.0 / first["decode_tok_s"], dtype="bf16", clocks=clk, gpu_launches=launches, sizes=out,
+              e2e={"value": first["decode_tok_s"], "unit": "tok/s", "h2d_bytes_per_step": 0, "d2h_bytes_per_step": 4,
+                   "note": "device loop: token ids stay on the device, 4 bytes per token come back"},
+              config=dict(base["config"], workload="Desalorn at model-like sizes beside the equal-size Fegizen and Fapudra stacks", context=CONTEXT,
+                          l2="inputs larger than L2 (weights streamed per token)")))
+
+
 def run(args, base, emit, write_yalm, shm_path, ClockSampler):
     import torch
     from yalm_b200 import api
