@@ -638,7 +638,7 @@ __global__ void glu_act_rows_kernel(float *__restrict__ h, const float *__restri
 // differ; a sum of two or more experts adds their scores).  Every expert finds its own place: the number of experts before it.  One
 // CTA per row; E <= 1024.
 template <int DT>
-__global__ void __launch_bounds__(256) router_topk_rows_kernel(int *__restrict__ ids, float *__restrict__ wts, const float *__restrict__ x, int ldx,
+__global__ void __launch_bounds__(1024) router_topk_rows_kernel(int *__restrict__ ids, float *__restrict__ wts, const float *__restrict__ x, int ldx,
                                                                const void *__restrict__ wr, int E, int top, int dim, int score, int renorm,
                                                                float renorm_eps, int groups, int keep, int group_top, bool vec,
                                                                const float *__restrict__ bias, float wscale) {
@@ -1031,7 +1031,8 @@ extern "C" int yalm_router_group_topk_rows(int *ids, float *wts, const float *x,
 	    keep_groups > groups || top > keep_groups * (n_experts / groups))
 		return YALM_EINVAL;
 	const bool vec = row_vec(wr, dim, dtype) && aligned16(x) && ldx % 4 == 0;
-	DISPATCH_DT(dtype, (router_topk_rows_kernel<DT><<<n, n <= 4 ? 256 : 128, sizeof(float) * (2 * n_experts + groups + top), (cudaStream_t)s>>>(
+	const int threads = n <= 4 ? std::min(1024, std::max(256, 32 * n_experts)) : 128; // a decode row: one warp per expert
+	DISPATCH_DT(dtype, (router_topk_rows_kernel<DT><<<n, threads, sizeof(float) * (2 * n_experts + groups + top), (cudaStream_t)s>>>(
 	                       ids, wts, x, ldx, wr, n_experts, top, dim, score, renorm, renorm_eps, groups, keep_groups, group_top, vec, bias, weight_scale)));
 	return (int)cudaGetLastError();
 }

@@ -498,6 +498,7 @@ struct GroupNormArgs {
 	const float *w;
 	int groups, dim;
 	float eps;
+	int vec; // rows are 16-byte aligned multiples of four channels
 };
 __global__ void __launch_bounds__(1024) group_norm_rows_kernel(GroupNormArgs g) {
 	extern __shared__ __align__(16) float gn_sm[]; // dim values, then partial sums of squares
@@ -506,19 +507,41 @@ __global__ void __launch_bounds__(1024) group_norm_rows_kernel(GroupNormArgs g) 
 	float *xr = g.x + (size_t)(g.rows ? g.rows[m] : m) * dim;
 	const bool add = g.a || g.b || g.y;
 	const size_t o = (size_t)m * dim;
-#pragma unroll 4
-	for (int e = tid; e < dim; e += nt) {
-		float v = xr[e];
-		if (add) {
-			float s = g.a ? g.a[o + e] : 0.f, f = 0.f;
-			if (g.abias) s += g.abias[e];
-			if (g.b) s += g.b[o + e];
-			for (int j = 0; j < g.nsum; ++j) f += g.y[((size_t)m * g.nsum + j) * g.ldy + e];
-			v = fmaf(g.mult, s + f, v);
-			xr[e] = v;
+	if (g.vec) {
+		// every operand of a piece of four channels is on its way before the first is used: one memory round trip
+		constexpr int U = 4;
+		const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+		auto get = [&](const float *p) { return *reinterpret_cast<const float4 *>(p); };
+		auto plus = [](float4 p, float4 q) { return make_float4(p.x + q.x, p.y + q.y, p.z + q.z, p.w + q.w); };
+		for (int e = tid * 4; e < dim; e += nt * 4) {
+			float4 v = get(xr + e);
+			if (add) {
+				const float *y = g.y + (size_t)m * g.nsum * g.ldy + e;
+				const float4 a = g.a ? get(g.a + o + e) : zero, c = g.abias ? get(g.abias + e) : zero, b = g.b ? get(g.b + o + e) : zero;
+				float4 f[U];
+#pragma unroll
+				for (int j = 0; j < U; ++j) f[j] = j < g.nsum ? get(y + (size_t)j * g.ldy) : zero;
+				float4 t = plus(plus(f[0], f[1]), plus(f[2], f[3]));
+				for (int j = U; j < g.nsum; ++j) t = plus(t, get(y + (size_t)j * g.ldy));
+				t = plus(plus(plus(a, c), b), t);
+				v = make_float4(fmaf(g.mult, t.x, v.x), fmaf(g.mult, t.y, v.y), fmaf(g.mult, t.z, v.z), fmaf(g.mult, t.w, v.w));
+				*reinterpret_cast<float4 *>(xr + e) = v;
+			}
+			*reinterpret_cast<float4 *>(vals + e) = v;
 		}
-		vals[e] = v;
-	}
+	} else
+		for (int e = tid; e < dim; e += nt) {
+			float v = xr[e];
+			if (add) {
+				float s = g.a ? g.a[o + e] : 0.f, f = 0.f;
+				if (g.abias) s += g.abias[e];
+				if (g.b) s += g.b[o + e];
+				for (int j = 0; j < g.nsum; ++j) f += g.y[((size_t)m * g.nsum + j) * g.ldy + e];
+				v = fmaf(g.mult, s + f, v);
+				xr[e] = v;
+			}
+			vals[e] = v;
+		}
 	if (!g.w) return;
 	__syncthreads();
 	const int size = dim / g.groups, wpg = max(1, nw / g.groups), slots = nw / wpg; // warps per group, groups in flight
@@ -537,6 +560,16 @@ __global__ void __launch_bounds__(1024) group_norm_rows_kernel(GroupNormArgs g) 
 	}
 	__syncthreads();
 	const float *r = part + g.groups * wpg;
+	if (g.vec && size % 4 == 0) {
+		for (int e = tid * 4; e < dim; e += nt * 4) {
+			const float4 v = *reinterpret_cast<const float4 *>(vals + e), w = *reinterpret_cast<const float4 *>(g.w + e);
+			const float k = r[e / size];
+			const float4 h = make_float4(v.x * k * w.x, v.y * k * w.y, v.z * k * w.z, v.w * k * w.w);
+			if (g.out) *reinterpret_cast<float4 *>(g.out + o + e) = h;
+			if (g.out16) *reinterpret_cast<uint2 *>(static_cast<uint16_t *>(g.out16) + o + e) = pack4_16(h, g.bf16);
+		}
+		return;
+	}
 	for (int e = tid; e < dim; e += nt) {
 		const float v = vals[e] * r[e / size] * g.w[e];
 		if (g.out) g.out[o + e] = v;
@@ -707,9 +740,10 @@ extern "C" int yalm_layer_norm_rows(float *out, void *out16, int bf16, float *x,
 	return (int)cudaGetLastError();
 }
 
-static int launch_group_norm(const GroupNormArgs &g, int n, cudaStream_t st) {
+static int launch_group_norm(GroupNormArgs g, int n, cudaStream_t st) {
 	if (!g.x || n < 1 || g.dim < 1 || g.groups < 1 || g.dim % g.groups || g.nsum < 0 || (g.nsum && !g.y) || (g.w && !g.out && !g.out16)) return YALM_EINVAL;
-	const int threads = n <= 4 && g.dim > 512 ? 1024 : 256;
+	g.vec = g.dim % 4 == 0 && g.ldy % 4 == 0 && al16(g.x) && al16(g.a) && al16(g.abias) && al16(g.b) && al16(g.y) && al16(g.out) && al16(g.w) && ((uintptr_t)g.out16 & 7) == 0;
+	const int threads = n <= 4 && g.dim > 512 ? std::min(1024, (g.vec ? g.dim / 4 + 31 : g.dim + 31) / 32 * 32) : 256;
 	const size_t smem = sizeof(float) * ((size_t)g.dim + 2 * (size_t)g.groups + threads / 32);
 	if ((int)smem > device_info().max_smem_optin) return YALM_EINVAL;
 	if (smem > 48 * 1024) YALM_TRY(cudaFuncSetAttribute(group_norm_rows_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));

@@ -152,7 +152,8 @@ __global__ void norm_conv_state_kernel(float *state, const float *__restrict__ h
 // ---- latent attention: norms, rotation, cache append ----------------------------------------------------------------------
 // Row m of the packed projection P (ld): [o_q, +q_rank) the query latent: RMS norm with weight qw in place.  With a cache of
 // its own, [o_kv, +kv_rank) RMS-normed with weight kw is the key / value latent and [o_kv + kv_rank, +rot_dim) the shared key
-// part, whose first rot_dims channels are rotated; both go to the ring row (slot p % ring) as [latent | key part].
+// part, whose first rot_dims channels are rotated; both go to the ring row (slot p % ring) as [latent | key part].  grid (rows, 2):
+// the query latent and the cache row are CTAs of their own.
 template <typename CT>
 __global__ void __launch_bounds__(256) latent_post_rows_kernel(float *__restrict__ P, int ld, int o_q, int q_rank, const float *__restrict__ qw, int o_kv,
                                                                int kv_rank, int rot_dim, const float *__restrict__ kw, CT *__restrict__ ring_buf, int ring,
@@ -161,12 +162,14 @@ __global__ void __launch_bounds__(256) latent_post_rows_kernel(float *__restrict
 	__shared__ float red[33];
 	const int m = blockIdx.x, p = first_pos(ctl, pos0) + m;
 	float *row = P + (size_t)m * ld;
-	if (q_rank > 0) { // 0: the queries are projected at full rank, there is no query latent
+	if (blockIdx.y == 0) {
+		if (q_rank < 1) return; // the queries are projected at full rank, there is no query latent
 		float ss = 0.f;
 		for (int e = threadIdx.x; e < q_rank; e += blockDim.x) ss += row[o_q + e] * row[o_q + e];
 		ss = block_sum(ss, red);
 		const float r = 1.0f / sqrtf(ss / q_rank + eps);
 		for (int e = threadIdx.x; e < q_rank; e += blockDim.x) row[o_q + e] = row[o_q + e] * r * qw[e];
+		return;
 	}
 	if (!ring_buf) return;
 	float ss = 0.f;
@@ -527,11 +530,14 @@ __global__ void __launch_bounds__(kLaWarps * 32) attn_latent_rows_kernel(float *
 		if (pr && lane == 0) pr[dv] = M, pr[dv + 1] = L;
 	}
 }
-// out[m, h, :] = sum_z w_z acc_z / sum_z w_z L_z with w_z = exp(M_z - max M), splits taken in order (a split without keys has
-// M = -inf and no weight); with a gate (one number per row and head) times sigmoid(gate).  grid (heads, rows).
-__global__ void attn_latent_merge_kernel(float *__restrict__ out, int ldo, const float *__restrict__ part, int n_heads, int dv, int nsplit,
-                                         const float *__restrict__ sink, const float *__restrict__ gate = nullptr, int ldg = 0) {
-	__shared__ float wz[128]; // the splits' weights over the common sum (nsplit <= 128)
+// out[m, h, :] = sum_z w_z acc_z / sum_z w_z L_z with w_z = exp(M_z - max M) (a split without keys has M = -inf and no weight); with a
+// gate (one number per row and head) times sigmoid(gate).  The order of the sums is fixed by the number of splits.  grid (heads, rows,
+// pieces of 128 / SG channels), 128 threads: SG of them share a channel's splits (many splits: more loads in flight per channel).
+template <int SG>
+__global__ void __launch_bounds__(128) attn_latent_merge_kernel(float *__restrict__ out, int ldo, const float *__restrict__ part, int n_heads, int dv, int nsplit,
+                                                                const float *__restrict__ sink, const float *__restrict__ gate, int ldg) {
+	constexpr int CH = 128 / SG;
+	__shared__ float wz[128], os[SG > 1 ? 128 : 1]; // the splits' weights over the common sum (nsplit <= 128)
 	const int h = blockIdx.x, m = blockIdx.y;
 	const float *pr = part + (size_t)(m * n_heads + h) * nsplit * (dv + 2);
 	if (threadIdx.x < 32) { // lane = split (and split + 32, + 64, + 96)
@@ -544,26 +550,36 @@ __global__ void attn_latent_merge_kernel(float *__restrict__ out, int ldo, const
 			lz[k] = z < nsplit ? pr[(size_t)z * (dv + 2) + dv + 1] : 0.f;
 		}
 		const float M = warp_max(fmaxf(fmaxf(mz[0], mz[1]), fmaxf(mz[2], mz[3])));
-		float e[4], t[4];
+		float e[4], t = 0.f;
 #pragma unroll
-		for (int k = 0; k < 4; ++k) e[k] = mz[k] == -INFINITY ? 0.f : expf(mz[k] - M), t[k] = e[k] * lz[k];
-		// the sum runs over the splits in order
-		float L = 0.f;
-		for (int z = 0; z < nsplit; ++z) L += __shfl_sync(kFull, z < 32 ? t[0] : z < 64 ? t[1] : z < 96 ? t[2] : t[3], z & 31);
-		float fin = softmax_finish(M, L, sink, h);
+		for (int k = 0; k < 4; ++k) e[k] = mz[k] == -INFINITY ? 0.f : expf(mz[k] - M), t += e[k] * lz[k];
+		float fin = softmax_finish(M, warp_sum(t), sink, h);
 		if (gate) fin /= 1.0f + expf(-gate[(size_t)m * ldg + h]);
 #pragma unroll
 		for (int k = 0; k < 4; ++k)
 			if (lane + 32 * k < nsplit) wz[lane + 32 * k] = e[k] * fin;
 	}
+	const int c = blockIdx.z * CH + threadIdx.x % CH, sg = threadIdx.x / CH;
 	__syncthreads();
-	// grid.z cuts the channels: a thread's loads over the splits are independent, and more CTAs keep more of them in flight
-	for (int c = blockIdx.z * blockDim.x + threadIdx.x; c < dv; c += gridDim.z * blockDim.x) {
-		float o = 0.f;
+	float o = 0.f;
+	if (c < dv)
 #pragma unroll 16
-		for (int z = 0; z < nsplit; ++z) o = fmaf(wz[z], pr[(size_t)z * (dv + 2) + c], o);
-		out[(size_t)m * ldo + (size_t)h * dv + c] = o;
+		for (int z = sg; z < nsplit; z += SG) o = fmaf(wz[z], pr[(size_t)z * (dv + 2) + c], o);
+	if constexpr (SG > 1) {
+		os[threadIdx.x] = o;
+		__syncthreads();
+		if (sg) return;
+		o = 0.f;
+#pragma unroll
+		for (int k = 0; k < SG; ++k) o += os[k * CH + threadIdx.x];
 	}
+	if (c < dv) out[(size_t)m * ldo + (size_t)h * dv + c] = o;
+}
+static int launch_latent_merge(float *out, int ldo, const float *part, int n, int n_heads, int dv, int nsplit, const float *sink, const float *gate, int ldg,
+                               cudaStream_t st) {
+	if (nsplit <= 8 || n > 16) attn_latent_merge_kernel<1><<<dim3(n_heads, n, (dv + 127) / 128), 128, 0, st>>>(out, ldo, part, n_heads, dv, nsplit, sink, gate, ldg);
+	else attn_latent_merge_kernel<4><<<dim3(n_heads, n, (dv + 31) / 32), 128, 0, st>>>(out, ldo, part, n_heads, dv, nsplit, sink, gate, ldg);
+	return (int)cudaGetLastError();
 }
 
 // out[r] = layer norm (or RMS norm) of x[rows[r]] times w   (rows null: r itself)
@@ -639,10 +655,10 @@ extern "C" int yalm_latent_post_rows(float *proj, int ld, int o_q, int q_rank, c
 		return YALM_EINVAL;
 	cudaStream_t st = (cudaStream_t)s;
 	if (cache_f32)
-		latent_post_rows_kernel<float><<<n, 256, 0, st>>>(proj, ld, o_q, q_rank, q_norm, o_kv, kv_rank, rot_dim, kv_norm, (float *)ring_buf, ring, freq, magnitude,
+		latent_post_rows_kernel<float><<<dim3(n, 2), 256, 0, st>>>(proj, ld, o_q, q_rank, q_norm, o_kv, kv_rank, rot_dim, kv_norm, (float *)ring_buf, ring, freq, magnitude,
 		                                                  rot_dims, interleaved, eps, pos0, ctl);
 	else
-		latent_post_rows_kernel<__nv_bfloat16><<<n, 256, 0, st>>>(proj, ld, o_q, q_rank, q_norm, o_kv, kv_rank, rot_dim, kv_norm, (__nv_bfloat16 *)ring_buf, ring,
+		latent_post_rows_kernel<__nv_bfloat16><<<dim3(n, 2), 256, 0, st>>>(proj, ld, o_q, q_rank, q_norm, o_kv, kv_rank, rot_dim, kv_norm, (__nv_bfloat16 *)ring_buf, ring,
 		                                                          freq, magnitude, rot_dims, interleaved, eps, pos0, ctl);
 	return (int)cudaGetLastError();
 }
@@ -738,8 +754,8 @@ static int launch_attn_latent(float *out, int ldo, const float *q, int ldq, cons
 	attn_latent_rows_kernel<R, NP><<<dim3((n_heads + R - 1) / R, n, nsplit), kLaWarps * 32, smem, st>>>(out, ldo, q, ldq, (const __nv_bfloat16 *)rows, ld,
 	                                                                                                  nsplit > 1 ? ws : nullptr, n_heads, dk, dv, ring,
 	                                                                                                  window, scale, pos0, ctl, sink);
-	if (nsplit > 1) attn_latent_merge_kernel<<<dim3(n_heads, n, (dv + 127) / 128), 128, 0, st>>>(out, ldo, ws, n_heads, dv, nsplit, sink);
-	return (int)cudaGetLastError();
+	if (int rc = (int)cudaGetLastError()) return rc;
+	return nsplit > 1 ? launch_latent_merge(out, ldo, ws, n, n_heads, dv, nsplit, sink, nullptr, 0, st) : 0;
 }
 
 // Attention of n query rows (n_heads x dk each) over cached bf16 rows shared by all heads: key = the row's dk channels, value =
@@ -775,8 +791,7 @@ extern "C" int yalm_attn_latent_rows_sink(float *out, int ldo, const float *q, i
 extern "C" int yalm_attn_split_merge(float *out, int ldo, const float *part, int n, int n_heads, int dv, int nsplit, const float *sink, const float *gate,
                                      int ldg, yalm_stream_t s) {
 	if (!out || !part || n < 1 || n_heads < 1 || dv < 1 || nsplit < 1 || nsplit > 128) return YALM_EINVAL;
-	attn_latent_merge_kernel<<<dim3(n_heads, n, (dv + 127) / 128), 128, 0, (cudaStream_t)s>>>(out, ldo, part, n_heads, dv, nsplit, sink, gate, ldg);
-	return (int)cudaGetLastError();
+	return launch_latent_merge(out, ldo, part, n, n_heads, dv, nsplit, sink, gate, ldg, (cudaStream_t)s);
 }
 extern "C" int yalm_attn_latent_merge(float *out, int ldo, const float *part, int n, int n_heads, int dv, int nsplit, const float *sink, yalm_stream_t s) {
 	return yalm_attn_split_merge(out, ldo, part, n, n_heads, dv, nsplit, sink, nullptr, 0, s);
