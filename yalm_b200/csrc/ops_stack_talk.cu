@@ -19,6 +19,7 @@
 #include <cuda_bf16.h>
 
 #include <algorithm>
+#include <type_traits>
 
 namespace yalm {
 namespace stack {
@@ -305,7 +306,7 @@ __global__ void __launch_bounds__(kMdThreads) attn_mixed_decode_kernel(MixedArgs
 // grid (ceil(n / 16), ceil(H / HS), splits), 16 warps; a CTA computes every head's scores for its 16 rows and the outputs of HS heads.
 // Per tile of TK keys (all kv heads' keys and values at once):
 //   scores   a warp takes (head, 16 keys) products; scaled, capped and biased they go to Z (head, row, key) in shared memory
-//   mixing   a thread takes 8 heads x 4 keys of a row: sums over all heads' Z in registers, then back over Z's first HS planes
+//   mixing   a thread takes 8 heads x 2 keys of a row: sums over all heads' Z in registers, then back over Z's first HS planes
 //   sums     16 / HS warps per head: the online softmax of the head's rows (the same in each of them), then P V for the warp's DW
 //            value channels
 // Keys of the next tile load from the end of the scores on, its values from the end of the sums on.
@@ -373,21 +374,25 @@ __global__ void __launch_bounds__(kMmThreads) attn_mixed_mma_kernel(MixedArgs a,
 		__syncthreads();
 		const int base = lo_min + t * TK;
 		// ---- scores ----
-		for (int u = warp; u < H * (TK / 16); u += kMmWarps) {
-			const int h = u / (TK / 16), k0 = (u % (TK / 16)) * 16, g = h / R;
-			float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+		auto scores = [&](int h, int k0, auto pieces) { // NP products of 16 keys that share the query fragments
+			constexpr int NP = decltype(pieces)::value;
+			const int g = h / R;
+			float s[2 * NP][4];
+#pragma unroll
+			for (int x = 0; x < 2 * NP; ++x) s[x][0] = s[x][1] = s[x][2] = s[x][3] = 0.f;
 			const __nv_bfloat16 *qp = Qs + (size_t)(h * 16 + ar) * LDK + ac, *kp = Ks + (size_t)(g * TK + k0 + br) * LDK + bc;
 #pragma unroll 4
 			for (int d = 0; d < dk; d += 16) {
-				uint32_t A[4], B[4];
+				uint32_t A[4], B[NP][4];
 				mx_ldsm_x4(A, qp + d);
-				mx_ldsm_x4(B, kp + d);
-				mx_mma(s[0], A, B[0], B[1]);
-				mx_mma(s[1], A, B[2], B[3]);
+#pragma unroll
+				for (int x = 0; x < NP; ++x) mx_ldsm_x4(B[x], kp + (size_t)x * 16 * LDK + d);
+#pragma unroll
+				for (int x = 0; x < NP; ++x) mx_mma(s[2 * x], A, B[x][0], B[x][1]), mx_mma(s[2 * x + 1], A, B[x][2], B[x][3]);
 			}
 			const float *bh = a.bias ? a.bias + (size_t)h * a.n_bias : nullptr;
 #pragma unroll
-			for (int x = 0; x < 2; ++x)
+			for (int x = 0; x < 2 * NP; ++x)
 #pragma unroll
 				for (int half = 0; half < 2; ++half) {
 					const int r = (lane >> 2) + half * 8, key = k0 + x * 8 + (lane & 3) * 2, dist = p0 + i0 + r - base - key; // of the first of two keys
@@ -396,29 +401,30 @@ __global__ void __launch_bounds__(kMmThreads) attn_mixed_mma_kernel(MixedArgs a,
 					if (bh) v.x += __ldg(bh + min(max(dist, 0), a.n_bias - 1)), v.y += __ldg(bh + min(max(dist - 1, 0), a.n_bias - 1));
 					*reinterpret_cast<float2 *>(Z + ((size_t)h * 16 + r) * LDZ + key) = v;
 				}
-		}
+		};
+		if (H >= kMmWarps)
+			for (int h = warp; h < H; h += kMmWarps) scores(h, 0, std::integral_constant<int, TK / 16>());
+		else
+			for (int u = warp; u < H * (TK / 16); u += kMmWarps) scores(u / (TK / 16), (u % (TK / 16)) * 16, std::integral_constant<int, 1>());
 		__syncthreads();
 		if (t + 1 < t_end) stage(Ks, kc, dk, LDK, t + 1);
 		else asm volatile("cp.async.commit_group;" ::: "memory");
-		// ---- mixing: 8 heads x 4 keys of one row per thread ----
-		constexpr int QUADS = 16 * TK / 4; // (row, 4 keys)
-		const int mu = tid / QUADS, mq = tid % QUADS, mr = mq / (TK / 4), mk = (mq % (TK / 4)) * 4;
+		// ---- mixing: 8 heads x 2 keys of one row per thread ----
+		constexpr int PAIRS = 16 * TK / 2; // (row, 2 keys)
+		const int mu = tid / PAIRS, mq = tid % PAIRS, mr = mq / (TK / 2), mk = (mq % (TK / 2)) * 2;
 		const bool mixes = mu * 8 < HP;
-		float acc[8][4];
+		float acc[8][2];
 		if (mixes) {
 #pragma unroll
-			for (int x = 0; x < 8; ++x) acc[x][0] = acc[x][1] = acc[x][2] = acc[x][3] = 0.f;
+			for (int x = 0; x < 8; ++x) acc[x][0] = acc[x][1] = 0.f;
 			const float *zp = Z + (size_t)mr * LDZ + mk, *mp = Ms + mu * 8;
 #pragma unroll 4
 			for (int g = 0; g < H; ++g) {
-				const float4 v = *reinterpret_cast<const float4 *>(zp + (size_t)g * 16 * LDZ);
+				const float2 v = *reinterpret_cast<const float2 *>(zp + (size_t)g * 16 * LDZ);
 				const float4 wa = *reinterpret_cast<const float4 *>(mp + g * HP), wb = *reinterpret_cast<const float4 *>(mp + g * HP + 4);
 				const float w[8] = {wa.x, wa.y, wa.z, wa.w, wb.x, wb.y, wb.z, wb.w};
 #pragma unroll
-				for (int x = 0; x < 8; ++x) {
-					acc[x][0] = fmaf(w[x], v.x, acc[x][0]), acc[x][1] = fmaf(w[x], v.y, acc[x][1]);
-					acc[x][2] = fmaf(w[x], v.z, acc[x][2]), acc[x][3] = fmaf(w[x], v.w, acc[x][3]);
-				}
+				for (int x = 0; x < 8; ++x) acc[x][0] = fmaf(w[x], v.x, acc[x][0]), acc[x][1] = fmaf(w[x], v.y, acc[x][1]);
 			}
 		}
 		__syncthreads(); // every thread has its sums: the planes may be overwritten
@@ -427,10 +433,8 @@ __global__ void __launch_bounds__(kMmThreads) attn_mixed_mma_kernel(MixedArgs a,
 #pragma unroll
 			for (int x = 0; x < 8; ++x) {
 				if (mu * 8 + x >= nh) break;
-				float4 v;
-				v.x = key >= lo && key <= i ? acc[x][0] : -INFINITY, v.y = key + 1 >= lo && key + 1 <= i ? acc[x][1] : -INFINITY;
-				v.z = key + 2 >= lo && key + 2 <= i ? acc[x][2] : -INFINITY, v.w = key + 3 >= lo && key + 3 <= i ? acc[x][3] : -INFINITY;
-				*reinterpret_cast<float4 *>(Z + ((size_t)(mu * 8 + x) * 16 + mr) * LDZ + mk) = v;
+				*reinterpret_cast<float2 *>(Z + ((size_t)(mu * 8 + x) * 16 + mr) * LDZ + mk) =
+				    make_float2(key >= lo && key <= i ? acc[x][0] : -INFINITY, key + 1 >= lo && key + 1 <= i ? acc[x][1] : -INFINITY);
 			}
 		}
 		asm volatile("cp.async.wait_group 1;" ::: "memory"); // the tile's values
