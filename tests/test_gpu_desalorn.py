@@ -213,7 +213,7 @@ def mixed_case(T, H, G, dk, dv, rows=10, seed=0):
     return q, k, v, rng.standard_normal((rows, H)), np.eye(H) + 0.4 * rng.standard_normal((H, H)) / math.sqrt(H), 2.0 * rng.standard_normal((T, H))
 
 
-MIXED = [(4, 2, 16, 32, 10), (8, 2, 64, 64, 16), (3, 1, 32, 16, 7), (6, 6, 48, 80, 4), (16, 4, 128, 128, 32), (20, 4, 32, 48, 12), (1, 1, 16, 16, 2), (2, 1, 64, 128, 9)]
+MIXED = [(4, 2, 16, 32, 10), (8, 2, 64, 96, 18), (3, 1, 32, 16, 7), (6, 6, 48, 80, 4), (16, 4, 128, 128, 32), (20, 4, 32, 48, 12), (1, 1, 16, 16, 2), (2, 1, 64, 128, 9)]
 
 
 @pytest.mark.parametrize("route,sizes", [("rows32", [1]), ("rows32", [2, 50, 3]), ("rows16", [40, 1, 17]), ("decode", [1]), ("decode", [2, 5]), ("mma", [150]), ("mma", [16, 33, 20, 17])])
@@ -677,7 +677,7 @@ def test_serving_precision_generation_over_the_captured_step(tmp_path):
     cfg = O.make_config([
         ("attention", O.attention_mixer(heads=4, kv_heads=2, dim=32, vdim=32), O.moe_mlp(ff=32, experts=6, top=2, shared=32)),
         ("latent_attention", O.latent_mixer(heads=2, dim=32, rot_dim=32, vdim=32, kv_rank=64, q_rank=32, window=20), None),
-        ("retention", O.retention_mixer(heads=2, dim=32, vdim=32), O.moe_mlp(ff=32, experts=4, top=2, count=1, keep=1)),
+        ("retention", O.retention_mixer(heads=3, dim=32, vdim=40), O.moe_mlp(ff=32, experts=4, top=2, count=1, keep=1)),
     ], width=96, vocab=120)
     folder, W = checkpoint(tmp_path, cfg, seed=16)
     prompt, n = tokens_for(cfg, 40), 60
